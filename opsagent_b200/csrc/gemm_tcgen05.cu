@@ -28,6 +28,12 @@ static constexpr int UMMA_K = 16;
 static constexpr int GEMM_THREADS = 192;
 static constexpr int RASTER_GROUP_M = 16;
 
+OA_DEVINL float glu_row_scale(const GemmParams& p, int row) {
+    if (!p.row_scale) return 1.0f;
+    const int i = p.row_scale_idx[row];
+    return i >= 0 ? p.row_scale[i] : 0.0f;
+}
+
 template <int BN>
 struct GemmCfg {
     static constexpr int A_BYTES = BLOCK_M * BLOCK_K * 2;              // 16 KB
@@ -198,6 +204,11 @@ __global__ void __launch_bounds__(GEMM_THREADS) gemm_tcgen05_kernel(const __grid
                 if (row_ok && col0 < p.N) {
                     uint16_t* orow = reinterpret_cast<uint16_t*>(p.out) + (size_t)row * p.ldo + (col0 >> 1);
                     float f[16];
+                    if (p.glu_limit > 0.f) {
+                        const float sc = glu_row_scale(p, row);
+#pragma unroll
+                        for (int i = 0; i < 16; ++i) f[i] = clamped_glu_f32(__uint_as_float(v[i]) * sc, __uint_as_float(v[16 + i]) * sc, p.glu_limit, p.glu_slope);
+                    } else
 #pragma unroll
                     for (int i = 0; i < 16; ++i) {
                         float g = __uint_as_float(v[i]), u = __uint_as_float(v[16 + i]);
@@ -459,6 +470,11 @@ __global__ void __launch_bounds__(GEMM_THREADS, 1) gemm_persistent_kernel(const 
                         const float gg[8] = {g0.x, g0.y, g0.z, g0.w, g1.x, g1.y, g1.z, g1.w};
                         const float uu[8] = {u0.x, u0.y, u0.z, u0.w, u1.x, u1.y, u1.z, u1.w};
                         float f[8];
+                        if (p.glu_limit > 0.f) {
+                            const float sc = row < p.M ? glu_row_scale(p, row) : 0.f;
+#pragma unroll
+                            for (int k = 0; k < 8; ++k) f[k] = clamped_glu_f32(gg[k] * sc, uu[k] * sc, p.glu_limit, p.glu_slope);
+                        } else
 #pragma unroll
                         for (int k = 0; k < 8; ++k) f[k] = __fdividef(gg[k], 1.0f + __expf(-gg[k])) * uu[k];
                         if (row < p.M && col0 < p.N) {

@@ -2,7 +2,7 @@
 // attention (a compressed key/value cache), a gated delta rule with per-channel decay, a Mamba-2 state-space layer, or windowed attention
 // over cached keys and values (sliding window with optional kept first tokens, one or two score maps per head, optional sink, output gate,
 // optionally reading another layer's cache), each beside a routed mixture-of-experts feed-forward, with an optional looped block that
-// re-injects the embedding.  Four designs are registered: "Ratasun" (one weight-only layer norm per layer, sigmoid group-limited router, SwiGLU
+// re-injects the embedding.  Five designs are registered: "Ratasun" (one weight-only layer norm per layer, sigmoid group-limited router, SwiGLU
 // experts), "Zurevik" (two RMS norms per layer, softmax over the chosen router logits, squared-ReLU experts, scaled embedding, soft-capped
 // logits) and "Rofizen" (norm after the sum: x <- norm(alpha x + sublayer(x)), mixer and feed-forward in sequence; mixers: gated linear
 // attention with a decay per key channel, retention with a fixed decay per head and rotate-half rotary, or causal soft-capped attention with
@@ -11,7 +11,11 @@
 // joined by learned coefficients (hyper-connections), a token shift in front of every mixer, a looped block without re-injection; mixers:
 // latent attention with a low-rank query, rotate-half rotary with YaRN-scaled frequencies, a sliding window, a sink and a per-channel output
 // gate, or causal grouped-query attention with projection biases, short convolutions on q / k / v, interleaved rotary, rotated values
-// and a sink; feed-forward: dense with the tanh form of GELU.
+// and a sink; feed-forward: dense with the tanh form of GELU.  "Petipel": sublayers in sequence with an RMS norm on either side of each
+// (x += m norm(sublayer(norm(x))), weights stored around zero); mixers: causal grouped-query attention without rotation (a learned bias per
+// head and distance bucket on the scores, a query temperature, values of unit RMS that later layers mix with the first layer's, a gate per
+// head), or HGRN2 (a recurrence that writes with the complement of its forget gate); feed-forward: dense with PolyNorm, or experts with a
+// clamped gated activation that are chosen by, and read their input times, a sigmoid score.
 // Every size and constant is read from the checkpoint folder's config.json; nothing here is specific to one checkpoint.
 #pragma once
 #include <cstdio>
@@ -27,22 +31,26 @@ namespace oa {
 
 enum HyMixer : int { HY_LATENT_ATTENTION = 0, HY_CHANNEL_DELTA = 1, HY_MAMBA2 = 2, HY_WINDOW_ATTENTION = 3, HY_LINEAR_ATTENTION = 4, HY_ATTENTION_BESIDE_MEMORY = 5 };
 enum HyNorm : int { HY_LAYER_NORM = 0, HY_RMS_NORM = 1 };
-enum HyRouterKind : int { HY_ROUTER_SIGMOID_GROUPS = 0, HY_ROUTER_SOFTMAX_CHOSEN = 1, HY_ROUTER_TOKEN_TABLE = 2 };   // weights: sigmoid scores renormalised and scaled / softmax over the chosen logits / a table row per token id, 1 / top each
+enum HyRouterKind : int { HY_ROUTER_SIGMOID_GROUPS = 0, HY_ROUTER_SOFTMAX_CHOSEN = 1, HY_ROUTER_TOKEN_TABLE = 2, HY_ROUTER_SIGMOID_CHOSEN = 3 };   // weights: sigmoid scores renormalised and scaled / softmax over the chosen logits / a table row per token id, 1 / top each / the chosen logits' sigmoids as they are
 // linear-attention recurrences over an fp32 state S[dim, vdim] per head, o_t = S_t^T q_t:
 //   channel decay: S_t = diag(a_t) S_(t-1) + k_t v_t^T, a_t = sigmoid(z_t)^(1 / tau) per key channel from a low-rank projection (gated linear attention)
 //   head decay:    S_t = decay_h S_(t-1) + k_t v_t^T with a fixed decay per head, rotate-half rotary on q and k (retention)
+//   forget write:  S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T, f_t = l + (1 - l) sigmoid(z_t) per key channel with a lower bound l; q = silu(.), no keys (HGRN2)
 //   matrix memory: S_t = exp(f + m_(t-1) - m_t) S_(t-1) + exp(i - m_t) k_t v_t^T with log gates i, f, a running maximum m and a normaliser n (xLSTM's mLSTM)
-enum HyLinearKind : int { HY_LIN_CHANNEL_DECAY = 0, HY_LIN_HEAD_DECAY = 1, HY_LIN_MATRIX_MEMORY = 2 };
+enum HyLinearKind : int { HY_LIN_CHANNEL_DECAY = 0, HY_LIN_HEAD_DECAY = 1, HY_LIN_MATRIX_MEMORY = 2, HY_LIN_FORGET_WRITE = 3 };
 enum HyLinearNorm : int { HY_LIN_NORM_HEAD_WEIGHT = 0, HY_LIN_NORM_NONE = 1, HY_LIN_NORM_ALL_WEIGHT = 2 };   // weight of the per-head RMS norm: [vdim] shared by heads / none / [heads * vdim]
 
 struct HyLinear {
     int kind = HY_LIN_CHANNEL_DECAY, heads = 0, dim = 0, vdim = 0;
     float tau = 1.f, gate_cap = 0.f, rot_base = 10000.f; int rot_dims = 0;
     std::vector<float> decay;             // head decay: one per head
-    int norm = HY_LIN_NORM_HEAD_WEIGHT, gate_silu = 1;      // output gate: silu (1) or sigmoid (0) of a projection, per channel
+    int norm = HY_LIN_NORM_HEAD_WEIGHT, gate_silu = 1;      // output gate: silu (1) or sigmoid (0) of a projection, per channel (forget write: no output gate)
     bool q_scaled = true, k_scaled = false;                  // dim^-1/2 on q, or on k (after the rotation)
 };
-enum HyExpertAct : int { HY_EXPERT_SWIGLU = 0, HY_EXPERT_RELU2 = 1, HY_EXPERT_GELU_TANH = 2 };     // down(silu(gate x) * up x) / down(relu(up x)^2) / down(gelu_tanh(up x))
+// down(silu(gate x) * up x) / down(relu(up x)^2) / down(gelu_tanh(up x)) / down(g sigmoid(slope g) (u + 1)) with g = min(gate x, limit), u = clamp(up x, -limit, limit) /
+// down(a N(z) + b N(z^2) + c N(z^3) + e) with z = up x and N(.) = unit RMS over the width (PolyNorm)
+enum HyExpertAct : int { HY_EXPERT_SWIGLU = 0, HY_EXPERT_RELU2 = 1, HY_EXPERT_GELU_TANH = 2, HY_EXPERT_CLAMPED_GLU = 3, HY_EXPERT_POLY_NORM = 4 };
+constexpr float HY_CLAMPED_GLU_SLOPE = 1.702f;
 enum HyRotLayout : int { HY_ROT_INTERLEAVED = 0, HY_ROT_HALVES = 1 };                         // channel 2i pairs with 2i + 1 / channel i with i + dims / 2
 // YaRN: with where(t) = dims ln(original / (2 pi t)) / (2 ln base), lo = max(floor(where(fast)), 0), hi = min(ceil(where(slow)), dims - 1) and
 // ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), frequency i is f_i / factor * ramp_i + f_i (1 - ramp_i); cos and sin carry the amplitude 0.1 ln(factor) + 1
@@ -55,6 +63,8 @@ struct HyMoe {
     float scale = 1.f;
     int router = HY_ROUTER_SIGMOID_GROUPS, act = HY_EXPERT_SWIGLU;
     bool dense = false;                   // one feed-forward for every token (no router, no experts): down(act(up h)), width ff
+    float limit = 0.f;                    // clamped gated activation
+    bool weight_on_input = false;         // the router's weight multiplies the expert's input, not its output
     int shared_ff = 0;                    // > 0: a shared expert of this width runs for every token, times sigmoid(w_sg . h)
 };
 
@@ -79,6 +89,10 @@ struct HyLayer {
     // windowed attention, optional parts: conv > 0: a short causal convolution (no bias, no activation) on every channel of q, k and v, right
     // after the projection; rot_dims > 0: rotary on the first rot_dims channels of every query / key head; v_rot: the value of position j is
     // cached turned by j over all vdim channels (pair m by j rot_base^(-2m / vdim)), a head's output at position i is turned back by -i
+    // bias_max > 0: a learned bias per head and distance bucket is added to the scaled score: with B table rows, distances below B / 2 have a row
+    // each, then a logarithmic scale up to bias_max, the last row beyond.  v_norm: a value head is cached divided by its RMS.  v_mix: every
+    // such layer but the first caches (1 - lambda) v + lambda v_first, v_first = the first such layer's cached value of the same token (v_first: its layer, -1: this is the first)
+    int bias_max = 0, v_norm = 0, v_mix = 0, v_first = -1;
     int q_rank = 0, rot_layout = HY_ROT_INTERLEAVED, v_rot = 0;
     HyRotScaling rot_scaling;
     HyLinear lin;                         // HY_LINEAR_ATTENTION, and the memory side of HY_ATTENTION_BESIDE_MEMORY (whose attention side uses the fields above)
@@ -102,6 +116,9 @@ struct HybridConfig {
     // token_shift: the mixer's input h_t (after the norm) is replaced by h_t + (h_(t-1) - h_t) * shift, h_(t-1) as it was before its own
     // replacement (zeros before the first token); every layer execution carries the last h of a sequence in its state slot.
     bool sequential = false, token_shift = false; int streams = 0;
+    // branch_norm (sequential designs): a sublayer's output passes a norm of its own before it joins the residual: x <- x + residual_mult norm_b(sublayer(norm(x))).
+    // norm_around_zero: the layers' and the final norm weights are stored as w - 1
+    bool branch_norm = false, norm_around_zero = false; float residual_mult = 1.f;
     bool loop_reinject = true;                          // a looped block re-injects the embedding before every pass (x <- W_in [x ; x0] + step[pass])
     std::vector<HyLayer> layers;
     int loop_start = 0, loop_stop = 0, loop_times = 0;    // times == 0: no looped block
@@ -138,6 +155,7 @@ struct HybridConfig {
         if (architecture == "Zurevik") return "zurevik";
         if (architecture == "Rofizen") return "rofizen";
         if (architecture == "Gosavik") return "gosavik";
+        if (architecture == "Petipel") return "petipel";
         return "";
     }
 
@@ -147,10 +165,14 @@ struct HybridConfig {
         HybridConfig c; c.dir = dir;
         c.arch = registry_key(j.str("architecture"));
         if (c.arch.empty()) throw std::runtime_error("config.json: unknown architecture '" + j.str("architecture") + "'");
-        const bool zu = c.arch == "zurevik", ro = c.arch == "rofizen", go = c.arch == "gosavik";
+        const bool zu = c.arch == "zurevik", ro = c.arch == "rofizen", go = c.arch == "gosavik", pe = c.arch == "petipel";
         if (go) {
             c.norm = HY_RMS_NORM; c.sequential = true; c.token_shift = true; c.loop_reinject = false;
             if (j.get("streams") && j.get("streams")->t == Json::Num) { c.streams = integer(j, "streams", "the model"); if (c.streams < 1 || c.streams > 8) throw std::runtime_error("config.json: streams must be 1 .. 8"); }
+        }
+        if (pe) {
+            c.norm = HY_RMS_NORM; c.sequential = true; c.branch_norm = true; c.norm_around_zero = true; c.loop_reinject = false;
+            c.residual_mult = (float)num(j, "residual_mult", "the model");
         }
         if (zu) { c.norm = HY_RMS_NORM; c.two_norms = true; }
         if (ro) { c.post_norm = true; c.post_alpha = (float)num(j, "postln_alpha", "the model"); }
@@ -203,7 +225,25 @@ struct HybridConfig {
                 if (const Json* mk = m.get("mask")) if (mk->t == Json::Obj) { l.window = integer(*mk, "size", "mask"); if (l.window < 1) throw std::runtime_error("config.json: mask.size must be at least 1"); }
                 if (l.kv_heads <= 0 || l.heads % l.kv_heads || l.dim <= 0 || l.vdim > 256 || (l.vdim & 1) || l.dim > 1024 || l.rot_dims < 0 || l.rot_dims > l.dim || (l.rot_dims & 1) || l.conv < 1 || l.conv > 16 || !(l.rot_base > 0.f))
                     throw std::runtime_error("config.json: bad attention sizes");
-            } else if (type == "attention" || type == "attention_2") {
+            } else if (pe && type == "attention") {
+                // causal grouped-query attention, no rotation: distance bias, query temperature, unit-RMS values mixed with the first such layer's, a gate per head
+                l.type = HY_WINDOW_ATTENTION;
+                l.heads = integer(m, "heads", type.c_str()); l.kv_heads = integer(m, "kv_heads", type.c_str()); l.dim = integer(m, "dim", type.c_str());
+                l.vdim = integer(m, "vdim", type.c_str()); l.scale = (float)num(m, "scale", type.c_str()); l.bias_max = integer(m, "bias_max", type.c_str());
+                l.window = 1 << 30; l.gate = HY_GATE_HEAD; l.v_norm = 1;
+                if (const Json* qt = m.get("q_temp")) if (qt->t == Json::Obj) { l.q_temp_coef = (float)num(*qt, "coef", "q_temp"); l.q_temp_every = integer(*qt, "every", "q_temp"); if (l.q_temp_every < 1) throw std::runtime_error("config.json: q_temp.every must be at least 1"); }
+                if (const Json* vm = m.get("v_mix")) l.v_mix = (vm->t == Json::Bool && vm->b) || (vm->t == Json::Num && vm->n != 0);
+                if (l.v_mix) for (int i = 0; i < (int)c.layers.size() && l.v_first < 0; ++i) if (c.layers[i].v_mix) {
+                    l.v_first = i;
+                    if (c.layers[i].kv_heads != l.kv_heads || c.layers[i].vdim != l.vdim) throw std::runtime_error("config.json: layers that mix values need the same kv_heads and vdim");
+                }
+                if (l.kv_heads <= 0 || l.heads % l.kv_heads || l.dim <= 0 || l.vdim > 256 || l.dim > 1024 || l.bias_max < 1 || l.bias_max > (1 << 22)) throw std::runtime_error("config.json: bad attention sizes");
+            } else if (pe && type == "hgrn2") {
+                l.type = HY_LINEAR_ATTENTION; HyLinear& n = l.lin;
+                n.heads = l.heads = integer(m, "heads", type.c_str()); n.dim = l.dim = integer(m, "dim", type.c_str()); n.vdim = l.vdim = integer(m, "vdim", type.c_str());
+                n.kind = HY_LIN_FORGET_WRITE; n.norm = HY_LIN_NORM_HEAD_WEIGHT; n.q_scaled = false;
+                if (n.dim <= 0 || n.dim > 768) throw std::runtime_error("config.json: bad linear-attention sizes");
+            } else if (!pe && (type == "attention" || type == "attention_2")) {
                 // "attention": differential (two score maps), query/key norm, kept first tokens, gate per channel;
                 // "attention_2": one map, projection biases, a sink per head, gate per head, optionally another layer's keys and values
                 const bool diff = type == "attention";
@@ -255,8 +295,8 @@ struct HybridConfig {
             const bool recurrent = l.type == HY_CHANNEL_DELTA || l.type == HY_MAMBA2;
             if (l.heads <= 0 || l.vdim <= 0 || (recurrent && (l.conv < 1 || l.conv > 16))) throw std::runtime_error("config.json: bad mixer sizes");
             const Json* mj = lj.get("mlp");
-            if (mj && mj->t == Json::Obj && (ro || go) && mj->str("kind") == "dense") {
-                l.moe.present = true; l.moe.dense = true; l.moe.act = go ? HY_EXPERT_GELU_TANH : HY_EXPERT_RELU2; l.moe.experts = 1; l.moe.top = 1;
+            if (mj && mj->t == Json::Obj && (ro || go || pe) && mj->str("kind") == "dense") {
+                l.moe.present = true; l.moe.dense = true; l.moe.act = pe ? HY_EXPERT_POLY_NORM : go ? HY_EXPERT_GELU_TANH : HY_EXPERT_RELU2; l.moe.experts = 1; l.moe.top = 1;
                 l.moe.ff = integer(*mj, "ff", "mlp");
                 if (l.moe.ff <= 0) throw std::runtime_error("config.json: bad feed-forward width");
             } else if (mj && mj->t == Json::Obj) {
@@ -264,7 +304,11 @@ struct HybridConfig {
                 const Json& r = obj(*mj, "router", "mlp");
                 l.moe.present = true; l.moe.ff = integer(obj(*mj, "expert", "mlp"), "ff", "expert");
                 l.moe.experts = integer(r, "experts", "router"); l.moe.top = integer(r, "top", "router");
-                if (zu) { l.moe.router = HY_ROUTER_SOFTMAX_CHOSEN; l.moe.act = HY_EXPERT_RELU2; }
+                if (pe) {
+                    l.moe.router = HY_ROUTER_SIGMOID_CHOSEN; l.moe.act = HY_EXPERT_CLAMPED_GLU; l.moe.weight_on_input = true; l.moe.limit = (float)num(obj(*mj, "expert", "mlp"), "limit", "expert");
+                    if (l.moe.ff <= 0 || !(l.moe.limit > 0.f)) throw std::runtime_error("config.json: bad expert sizes");
+                }
+                else if (zu) { l.moe.router = HY_ROUTER_SOFTMAX_CHOSEN; l.moe.act = HY_EXPERT_RELU2; }
                 else if (ro) {
                     l.moe.router = HY_ROUTER_TOKEN_TABLE;
                     if (const Json* sh = mj->get("shared")) if (sh->t == Json::Obj) { l.moe.shared_ff = integer(*sh, "ff", "shared"); if (l.moe.shared_ff <= 0) throw std::runtime_error("config.json: bad shared expert width"); }

@@ -859,7 +859,7 @@ __global__ void __launch_bounds__(128) hy_gated_norm_kernel(const float* o, int 
         const int c = c0 + i;
         float v = o[(long long)t * C + c] * dv;
         if (skip) v = fmaf(skip[c / skip_block], ldf(xs + (long long)t * ld_xs + c), v);
-        if (gate_before) { const float g = ldf(gate + (long long)t * ld_gate + c); v *= act ? siluf_(g) : sigmoidf_(g); }
+        if (gate && gate_before) { const float g = ldf(gate + (long long)t * ld_gate + c); v *= act ? siluf_(g) : sigmoidf_(g); }
         ss += v * v;
     }
     const float rr = 1.0f / sqrtf(block_sum(ss, red) / (float)group + eps);
@@ -867,7 +867,7 @@ __global__ void __launch_bounds__(128) hy_gated_norm_kernel(const float* o, int 
         const int c = c0 + i;
         float v = o[(long long)t * C + c] * dv;
         if (skip) v = fmaf(skip[c / skip_block], ldf(xs + (long long)t * ld_xs + c), v);
-        const float g = ldf(gate + (long long)t * ld_gate + c), ga = act ? siluf_(g) : sigmoidf_(g);
+        const float g = gate ? ldf(gate + (long long)t * ld_gate + c) : 0.f, ga = !gate ? 1.f : act ? siluf_(g) : sigmoidf_(g);
         if (gate_before) v *= ga;
         v = v * rr * (w ? w[c % wlen] : 1.f);
         if (!gate_before) v *= ga;
@@ -906,7 +906,7 @@ __global__ void __launch_bounds__(128) hy_gated_norm_warp_kernel(const float* __
         if (skip) { ld4(xs + (long long)t * ld_xs + c, x4);
 #pragma unroll
             for (int e = 0; e < 4; ++e) v[e] = fmaf(skip[(c + e) / skip_block], x4[e], v[e]); }
-        if (gate_before) { ld4(gate + (long long)t * ld_gate + c, g);
+        if (gate && gate_before) { ld4(gate + (long long)t * ld_gate + c, g);
 #pragma unroll
             for (int e = 0; e < 4; ++e) v[e] *= act ? siluf_(g[e]) : sigmoidf_(g[e]); }
 #pragma unroll
@@ -921,10 +921,10 @@ __global__ void __launch_bounds__(128) hy_gated_norm_warp_kernel(const float* __
         if (skip) { ld4(xs + (long long)t * ld_xs + c, x4);
 #pragma unroll
             for (int e = 0; e < 4; ++e) v[e] = fmaf(skip[(c + e) / skip_block], x4[e], v[e]); }
-        ld4(gate + (long long)t * ld_gate + c, g);
+        if (gate) ld4(gate + (long long)t * ld_gate + c, g);
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            const float ga = act ? siluf_(g[e]) : sigmoidf_(g[e]);
+            const float ga = !gate ? 1.f : act ? siluf_(g[e]) : sigmoidf_(g[e]);
             if (gate_before) v[e] *= ga;
             v[e] = v[e] * rr * (w ? w[(c + e) % wlen] : 1.f);
             if (!gate_before) v[e] *= ga;
@@ -988,7 +988,7 @@ __global__ void __launch_bounds__(128) hy_moe_router_kernel(HyRouter m, const fl
     if (lane < m.top) { idx[(long long)t * m.top + lane] = my_e; wgt[(long long)t * m.top + lane] = mine / (sum + 1e-20f) * m.scale; }
 }
 
-// one warp per token: z = logits + bias, the `top` largest logits (ties -> lower index), weights = softmax over the chosen ones
+// one warp per token: z = logits + bias, the `top` largest logits (ties -> lower index), weights = softmax over the chosen ones (kind 3: their sigmoids)
 __global__ void __launch_bounds__(128) hy_moe_router_softmax_kernel(HyRouter m, const float* logits, int ldz, const float* bias, int32_t* idx, float* wgt, int T) {
     HY_PDL();
     extern __shared__ float sm[];
@@ -1008,13 +1008,17 @@ __global__ void __launch_bounds__(128) hy_moe_router_softmax_kernel(HyRouter m, 
         if (lane == 0) ch[bi] = -INFINITY;
         __syncwarp();
     }
+    if (m.kind == 3) {
+        if (lane < m.top) { idx[(long long)t * m.top + lane] = my_e; wgt[(long long)t * m.top + lane] = sigmoidf_(mine); }
+        return;
+    }
     const float p = lane < m.top ? expf(mine - first) : 0.f;
     const float sum = warp_sum(p);
     if (lane < m.top) { idx[(long long)t * m.top + lane] = my_e; wgt[(long long)t * m.top + lane] = p / sum; }
 }
 
 template <typename TA>
-__global__ void __launch_bounds__(256) hy_moe_gate_up_kernel(const TA* h, int ldh, const TA* gu, int ldw, int W, int ff, int ffp, const int32_t* idx, int top, TA* act) {
+__global__ void __launch_bounds__(256) hy_moe_gate_up_kernel(HyExpertForm form, const TA* h, int ldh, const TA* gu, int ldw, int W, int ff, int ffp, const int32_t* idx, int top, TA* act) {
     HY_PDL();
     const int row = blockIdx.x, t = row / top, e = idx[row], warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int f = blockIdx.y * 8 + warp;
@@ -1025,7 +1029,11 @@ __global__ void __launch_bounds__(256) hy_moe_gate_up_kernel(const TA* h, int ld
         float g = 0.f, u = 0.f;
         for (int i = lane; i < W; i += 32) { const float x = ldf(hr + i); g = fmaf(x, ldf(wg + i), g); u = fmaf(x, ldf(wu + i), u); }
         g = warp_sum(g); u = warp_sum(u);
-        v = siluf_(g) * u;
+        if (form.kind == 2) {
+            const float sc = form.in_weight ? form.in_weight[row] : 1.f;
+            g = fminf(g * sc, form.limit); u = fminf(fmaxf(u * sc, -form.limit), form.limit);
+            v = g * sigmoidf_(form.slope * g) * (u + 1.f);
+        } else v = siluf_(g) * u;
     }
     if (lane == 0) stf(act + (long long)row * ffp + f, v);
 }
@@ -1058,9 +1066,9 @@ __global__ void __launch_bounds__(256) hy_moe_down_kernel(const TA* act, const T
         float d = 0.f;
         for (int i = lane; i < ffp; i += 32) d = fmaf(ldf(ar + i), ldf(wd + i), d);
         d = warp_sum(d);
-        acc = fmaf(wgt[(long long)t * top + c], d, acc);
+        acc = fmaf(wgt ? wgt[(long long)t * top + c] : 1.f, d, acc);
     }
-    if (lane == 0) x[(long long)t * W + n] = fmaf(beta, x[(long long)t * W + n], acc);
+    if (lane == 0) x[(long long)t * W + n] = beta == 0.f ? acc : fmaf(beta, x[(long long)t * W + n], acc);
 }
 
 // Expert plan in three small kernels: (1) pairs per expert, (2) one CTA lays the experts' 128-row tiles out one after the other, (3) every
@@ -1142,11 +1150,12 @@ __global__ void hy_moe_combine_kernel(const float* y, int ldy, const int32_t* ds
     for (int c = threadIdx.x * 4; c < W; c += blockDim.x * 4) {
         float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
         for (int k = 0; k < top; ++k) {
-            const float w = wgt[(long long)t * top + k];
+            const float w = wgt ? wgt[(long long)t * top + k] : 1.f;
             const float4 v = *reinterpret_cast<const float4*>(y + (long long)dst_of[(long long)t * top + k] * ldy + c);
             acc.x = fmaf(w, v.x, acc.x); acc.y = fmaf(w, v.y, acc.y); acc.z = fmaf(w, v.z, acc.z); acc.w = fmaf(w, v.w, acc.w);
         }
         float4* xp = reinterpret_cast<float4*>(x + (long long)t * W + c);
+        if (beta == 0.f) { *xp = acc; continue; }
         float4 xv = *xp; xv.x = fmaf(beta, xv.x, acc.x); xv.y = fmaf(beta, xv.y, acc.y); xv.z = fmaf(beta, xv.z, acc.z); xv.w = fmaf(beta, xv.w, acc.w); *xp = xv;
     }
 }
@@ -1391,13 +1400,13 @@ cudaError_t hy_moe_router_softmax(const HyRouter& m, const float* logits, int ld
     if (m.top > 32) return cudaErrorInvalidValue;
     return launch_plain(hy_moe_router_softmax_kernel, dim3((T + 3) / 4), dim3(128), (size_t)4 * m.experts * 4, s, m, logits, ldz, bias, idx, wgt, T);
 }
-cudaError_t hy_moe_gate_up(bool f32, int relu2, const void* h, int ldh, const void* gu, int ldw, int W, int ff, int ffp, const int32_t* idx, int top, void* act, int T, cudaStream_t s) {
+cudaError_t hy_moe_gate_up(bool f32, const HyExpertForm& form, const void* h, int ldh, const void* gu, int ldw, int W, int ff, int ffp, const int32_t* idx, int top, void* act, int T, cudaStream_t s) {
     dim3 grid(T * top, (ffp + 7) / 8);
-    if (relu2)
+    if (form.kind == 1)
         return f32 ? launch_plain(hy_moe_up_relu2_kernel<float>, grid, dim3(256), 0, s, (const float*)h, ldh, (const float*)gu, ldw, W, ff, ffp, idx, top, (float*)act)
                    : launch_plain(hy_moe_up_relu2_kernel<bf>, grid, dim3(256), 0, s, (const bf*)h, ldh, (const bf*)gu, ldw, W, ff, ffp, idx, top, (bf*)act);
-    return f32 ? launch_plain(hy_moe_gate_up_kernel<float>, grid, dim3(256), 0, s, (const float*)h, ldh, (const float*)gu, ldw, W, ff, ffp, idx, top, (float*)act)
-               : launch_plain(hy_moe_gate_up_kernel<bf>, grid, dim3(256), 0, s, (const bf*)h, ldh, (const bf*)gu, ldw, W, ff, ffp, idx, top, (bf*)act);
+    return f32 ? launch_plain(hy_moe_gate_up_kernel<float>, grid, dim3(256), 0, s, form, (const float*)h, ldh, (const float*)gu, ldw, W, ff, ffp, idx, top, (float*)act)
+               : launch_plain(hy_moe_gate_up_kernel<bf>, grid, dim3(256), 0, s, form, (const bf*)h, ldh, (const bf*)gu, ldw, W, ff, ffp, idx, top, (bf*)act);
 }
 cudaError_t hy_moe_down(bool f32, const void* act, const void* down, int W, int ffp, const int32_t* idx, const float* wgt, int top, float* x, int T, cudaStream_t s, float beta) {
     dim3 grid(T, (W + 7) / 8);

@@ -66,7 +66,16 @@ cudaError_t hy_post_norm(bool f32, float* x, float beta, const float* y1, const 
 // out_rot (1: pairs 2m / 2m + 1, 2: pairs m / m + vdim / 2): every head's output at position i is turned by -i over all vdim channels with the
 // angles of out_cos / out_sin ([position, vdim / 2]) before the gate: the counterpart of values that were cached turned by their own position.
 struct HyWinAttn { int heads, kv_heads, dim, vdim, maps, window, keep_first, qk_norm, gate; float scale, lambda, out_scale; float softcap = 0.f, slope_exp = 0.f, q_temp_coef = 0.f; int q_temp_every = 0;
-                   int out_rot = 0; const float* out_cos = nullptr; const float* out_sin = nullptr; };
+                   int out_rot = 0; const float* out_cos = nullptr; const float* out_sin = nullptr;
+                   // rel != null: head h's scaled score with a key at distance n gains rel[h * rel_len + min(n, rel_len - 1)] (fp32); rel_run[n] = the
+                   // largest distance up to which every entry from n on is the same row of the bias table (beyond the table: INT_MAX).
+                   // With rel, the query temperature multiplies the scores (fp32) instead of the stored queries
+                   const float* rel = nullptr; const int32_t* rel_run = nullptr; int rel_len = 0; };
+// Preparation of a layer with unit-RMS values (maps = 1, queries as they are): keys go to cache row slots[t] unchanged; every value head is divided by
+// sqrt(mean(v^2) + eps) and, with first != null, becomes (1 - lambda) v + lambda v_first before it is cached, v_first = the same token's cached value
+// in another layer's cache `first` (row width first_row, values from column first_col on)
+struct HyValueMix { const void* first; int first_row, first_col; float lambda; };
+cudaError_t hy_win_value_prep(bool f32, const HyWinAttn& a, const void* k, const void* v, int ldkv, const HyValueMix& mix, float eps, void* cache, const HyRows& r, cudaStream_t s);
 // Rotary preparation of a cached-key/value attention layer (maps = 1, no query / key norm): the first rot_dims channels of every query head (in
 // place) and key head turn by the row's position (layout 0: pairs 2i / 2i + 1, 1: pairs i / i + rot_dims / 2; tables [position, rot_dims / 2]);
 // with v_cos / v_sin ([position, vdim / 2]) every value head turns over all of its channels in the same layout; keys and values go to cache row slots[t].
@@ -174,6 +183,10 @@ struct HyLinPrep { int heads, dim, vdim; bool q_scaled, k_scaled; int rot_dims; 
 // channel decay (z != null): dec[t, h, d] = sigmoid(z[t, h, d])^(1 / tau) = exp(logsigmoid(z) / tau), in place on the fp32 z (= dec);  head decay: dec[t, h] = decay[h]
 cudaError_t hy_lin_prep(bool f32, const HyLinPrep& p, const void* q, const void* k, const void* v, int ld, float* qq, float* kk, float* vv, float* dec_channel, float tau,
                         const float* decay_head, float* dec_head, const float* rope_cos, const float* rope_sin, const HyRows& r, cudaStream_t s);
+// Forget write: q [T, ld] -> qq = silu(q), z [T, ld] -> dec = f = lower + (1 - lower) sigmoid(z + bias) and kk = 1 - f = (1 - lower) sigmoid(-(z + bias))
+// (its own evaluation: no cancellation where the gate is nearly open), v -> vv; lower, bias [heads * dim] fp32
+cudaError_t hy_forget_prep(bool f32, int heads, int dim, int vdim, const void* q, const void* z, const void* v, int ld, const float* bias, const float* lower, float* qq, float* kk, float* vv,
+                           float* dec, int T, cudaStream_t s);
 // Matrix memory.  gates [T, ldg] fp32 = [W_i h + b_i | W_f h + b_f] (heads each).  hy_mlstm_gates: log gates i = cap tanh(. / cap),
 // f = logsigmoid(cap tanh(. / cap)); the running maximum m_t = max(f_t + m_(t-1), i_t) per (sequence, head), carried in mstate [slots, heads]
 // (a sequence whose step starts at position 0 starts from m = 0); out: dec[t, h] = exp(f + m_(t-1) - m_t), gin[t, h] = exp(i - m_t), floor_[t, h] = exp(-m_t)
@@ -182,25 +195,29 @@ cudaError_t hy_mlstm_gates(const float* gates, int ldg, int heads, float cap, fl
 cudaError_t hy_mlstm_prep(bool f32, int heads, int dim, int vdim, const void* q, const void* k, const void* v, int ld, const float* gin, float* qq, float* kk, float* vv, int T, cudaStream_t s);
 // group-wise RMS norm with a gate: v = o (+ skip[c / skip_block] * xs[t, c]); gate_before ? v *= act(gate) : -; v /= rms over each group of
 // `group` channels; v *= w[c % wlen]; !gate_before ? v *= act(gate) : -.  act: 0 = sigmoid, 1 = silu.
-// w == null: no weight.  den_dot != null: every group's o is first divided by max(|den_dot[t, g]|, den_floor[t, g]) + 1e-6 (the matrix memory's normaliser)
+// w == null: no weight.  gate == null: no gate.  den_dot != null: every group's o is first divided by max(|den_dot[t, g]|, den_floor[t, g]) + 1e-6 (the matrix memory's normaliser)
 cudaError_t hy_gated_norm(bool f32, const float* o, int C, int group, const float* w, int wlen, const void* gate, int ld_gate, int gate_before, int act,
                           const float* skip, int skip_block, const void* xs, int ld_xs, void* out, int ld_out, float eps, int T, cudaStream_t s,
                           const float* den_dot = nullptr, const float* den_floor = nullptr);
 
-struct HyRouter { int experts, top, groups, keep; float scale; int kind; };     // kind 0: the sigmoid router below; 1: hy_moe_router_softmax
+struct HyRouter { int experts, top, groups, keep; float scale; int kind; };     // kind 0: the sigmoid router below; 1, 3: hy_moe_router_softmax
 // sigmoid router over fp32 logits [T, ldz] with a selection-only correction and group-limited choice: a group's score is the sum of its two
 // largest corrected scores, only the best `keep` groups compete; idx[t, top], wgt[t, top] = chosen uncorrected sigmoids / their sum * scale
 cudaError_t hy_moe_router(const HyRouter& m, const float* logits, int ldz, const float* correction, int32_t* idx, float* wgt, int T, cudaStream_t s);
-// router whose weights are the softmax over the chosen logits only: z = logits + bias (fp32), the `top` largest (ties -> lower index), wgt = softmax of those
+// router whose weights are the softmax over the chosen logits only: z = logits + bias (fp32), the `top` largest (ties -> lower index), wgt = softmax of those;
+// kind 3: wgt = sigmoid(z) of the chosen, as they are
 cudaError_t hy_moe_router_softmax(const HyRouter& m, const float* logits, int ldz, const float* bias, int32_t* idx, float* wgt, int T, cudaStream_t s);
 // router without scores: token id -> its `top` experts from table [vocab, top], weight 1 / top each.  shared >= 0: one more choice for every
 // token, expert `shared` with weight sigmoid(w_sg . h[t]) (fp32 sum).  idx / wgt: [T, top (+ 1)]
 cudaError_t hy_moe_router_table(bool f32, const int32_t* tokens, const int32_t* table, int vocab, int top, int shared, const void* h, int ldh, const void* w_sg, int W,
                                 int32_t* idx, float* wgt, int T, cudaStream_t s);
-// routed experts, one (token, choice) at a time (decode-sized batches and the fp32 mode).  relu2 == 0: SwiGLU, gu: [E][2 ffp][ldw] with gate / up
-// rows interleaved in blocks of 16; relu2 == 1: act = relu(up h)^2, gu: [E][ffp][ldw] (up rows only).  down: [E][W][ffp]; act: [T * top, ffp]
-cudaError_t hy_moe_gate_up(bool f32, int relu2, const void* h, int ldh, const void* gu, int ldw, int W, int ff, int ffp, const int32_t* idx, int top, void* act, int T, cudaStream_t s);
-// x[t] = beta * x[t] + sum over choices
+// routed experts, one (token, choice) at a time (decode-sized batches and the fp32 mode).  kind 0: SwiGLU, gu: [E][2 ffp][ldw] with gate / up
+// rows interleaved in blocks of 16; kind 1: act = relu(up h)^2, gu: [E][ffp][ldw] (up rows only); kind 2: the clamped gated activation
+// g sigmoid(slope g) (u + 1), g = min(gate x, limit), u = clamp(up x, -limit, limit), gu as in kind 0.  in_weight (kind 2; [T * top] or null): the
+// expert reads in_weight * h (the products are linear: the fp32 sums are scaled).  down: [E][W][ffp]; act: [T * top, ffp]
+struct HyExpertForm { int kind; float limit; float slope; const float* in_weight; };
+cudaError_t hy_moe_gate_up(bool f32, const HyExpertForm& form, const void* h, int ldh, const void* gu, int ldw, int W, int ff, int ffp, const int32_t* idx, int top, void* act, int T, cudaStream_t s);
+// x[t] = beta * x[t] + sum over choices of wgt * (.); wgt == null: weights 1; beta == 0: x is written only
 cudaError_t hy_moe_down(bool f32, const void* act, const void* down, int W, int ffp, const int32_t* idx, const float* wgt, int top, float* x, int T, cudaStream_t s, float beta = 1.f);
 
 // grouped (tensor-core) expert path: rows sorted by expert into 128-row tiles
@@ -208,7 +225,7 @@ cudaError_t hy_moe_down(bool f32, const void* act, const void* down, int W, int 
 // count at [0] and 2 * experts words of scratch from [4]
 cudaError_t hy_moe_plan(const int32_t* idx, int T, int top, int experts, int32_t* tile_expert, int32_t* row_src, int32_t* n_tiles_out, int32_t* dst_of, int max_tiles, cudaStream_t s);
 cudaError_t hy_moe_gather(const void* h, int ldh, int W, const int32_t* row_src, const int32_t* n_tiles, int top, void* out, int max_tiles, cudaStream_t s);
-// x[t] = beta * x[t] + sum over choices (in order) wgt[t,c] * y[dst_of[t*top+c]]
+// x[t] = beta * x[t] + sum over choices (in order) wgt[t,c] * y[dst_of[t*top+c]]; wgt == null: weights 1; beta == 0: x is written only
 cudaError_t hy_moe_combine(const float* y, int ldy, const int32_t* dst_of, const float* wgt, int top, float* x, int W, int T, cudaStream_t s, float beta = 1.f);
 
 // ---- several residual streams joined by learned coefficients (hyper-connections), token shift (hybrid_streams.cu) ----
@@ -229,6 +246,16 @@ cudaError_t hy_stream_norm(bool f32, const HyStreams& c, float* xs, const float*
 cudaError_t hy_token_shift(bool f32, const float* hn, const float* prev, const float* mu, void* h, int ldh, const HyRows& r, int W, cudaStream_t s);
 // out[t, :n] = in[t, :n] / sqrt(mean(in[t, :n]^2) + eps) * w — RMS norm of a projection's first n columns (fp32 arithmetic, activation type in and out)
 cudaError_t hy_rmsnorm_act(bool f32, const void* in, int ld_in, int n, const float* w, void* out, int ld_out, float eps, int T, cudaStream_t s);
+// z[t, :n] <- a N(z) + b N(z^2) + c N(z^3) + e in place (activation type, fp32 arithmetic), N(u) = u / sqrt(mean(u^2) + eps) over the n columns
+struct HyPolyCoef { float a, b, c, e; };
+cudaError_t hy_poly_norm(bool f32, void* z, int ldz, int n, const HyPolyCoef& k, float eps, int T, cudaStream_t s);
+// Plain residual whose sublayers' outputs pass a norm of their own: closes one sublayer and opens the next in one pass over the row, each part optional
+//  (1) b.y != null: x[t] <- x[t] + b.mult * (y / sqrt(mean(y^2) + eps) * b.w);  y = b.y[t] ([T, W] fp32), or with b.dst_of the sum over the row's b.top
+//      choices (in order) of b.y[b.dst_of[t * top + c]] (grouped experts: the rows of their sorted tiles)
+//  (2) w != null: h[t] = x / sqrt(mean(x^2) + eps) * w of the new x (activation type, pitch ldh).  rows != null: output row t reads row rows[t] of x
+//      and y, and x itself stays
+struct HyBranch { const float* y; const float* w; float mult; const int32_t* dst_of; int top; };
+cudaError_t hy_branch_norm(bool f32, float* x, const HyBranch& b, const int32_t* rows, const float* w, float eps, void* h, int ldh, int T, int W, cudaStream_t s);
 // x[t, c] *= sigmoid(g[t, c]) for c < n, in place (activation type)
 cudaError_t hy_sigmoid_gate(bool f32, void* x, int ldx, const void* g, int ldg, int n, int T, cudaStream_t s);
 

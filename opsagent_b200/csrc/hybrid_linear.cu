@@ -1,6 +1,6 @@
 // hybrid_linear.cu — kernels around the linear-attention recurrences of the hybrid decoder family (API: hybrid_kernels.hpp): operands of
-// gated linear attention (a decay per key channel), retention (a fixed decay per head, rotate-half rotary) and the xLSTM matrix memory (log
-// gates, running maximum, normaliser); the norm after the sum that closes a sublayer of a post-norm design; the router that reads a token's
+// gated linear attention (a decay per key channel), retention (a fixed decay per head, rotate-half rotary), HGRN2 (a forget gate with a lower
+// bound whose complement is what is written) and the xLSTM matrix memory (log gates, running maximum, normaliser); the norm after the sum that closes a sublayer of a post-norm design; the router that reads a token's
 // experts from a table.  The recurrences themselves are hy_recurrence (hybrid_kernels.cu).  Everything here is fp32 arithmetic; TA is the
 // element type of projection outputs and of the rows handed to the next matrix product.
 #include "hybrid_common.cuh"
@@ -259,6 +259,47 @@ __global__ void __launch_bounds__(128) hy_mlstm_prep_kernel(int H, int D, int VD
     for (int i = threadIdx.x; i < H * VD; i += blockDim.x) vv[t * H * VD + i] = ldf(v + t * ld + i);
 }
 
+// Operands of the recurrence that writes with the complement of its forget gate.  kk = 1 - f comes from sigmoid of the negated argument.
+__device__ __forceinline__ void forget_gate(float z, float lower, float& f, float& w) {
+    const float e = expf(-fabsf(z)), big = 1.0f / (1.0f + e), small = e * big, open = 1.0f - lower;      // sigmoid(|z|), sigmoid(-|z|)
+    f = fmaf(open, z >= 0.f ? big : small, lower); w = open * (z >= 0.f ? small : big);
+}
+template <typename TA>
+__global__ void __launch_bounds__(128) hy_forget_prep_kernel(int H, int D, int VD, const TA* __restrict__ q, const TA* __restrict__ z, const TA* __restrict__ v, int ld,
+                                                             const float* __restrict__ bias, const float* __restrict__ lower, float* __restrict__ qq, float* __restrict__ kk,
+                                                             float* __restrict__ vv, float* __restrict__ dec) {
+    HY_PDL();
+    const long long t = blockIdx.x;
+    for (int i = threadIdx.x; i < H * D; i += blockDim.x) {
+        float f, w; forget_gate(ldf(z + t * ld + i) + bias[i], lower[i], f, w);
+        qq[t * H * D + i] = siluf_(ldf(q + t * ld + i)); dec[t * H * D + i] = f; kk[t * H * D + i] = w;
+    }
+    for (int i = threadIdx.x; i < H * VD; i += blockDim.x) vv[t * H * VD + i] = ldf(v + t * ld + i);
+}
+// The same for bf16 rows in aligned groups of 8 channels: 16 bytes per access, the same bits
+__global__ void __launch_bounds__(128) hy_forget_prep_vec8_kernel(int nqk, int nv, const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ z,
+                                                                  const __nv_bfloat16* __restrict__ v, int ld, const float* __restrict__ bias, const float* __restrict__ lower,
+                                                                  float* __restrict__ qq, float* __restrict__ kk, float* __restrict__ vv, float* __restrict__ dec) {
+    HY_PDL();
+    const long long t = blockIdx.x;
+    for (int it = threadIdx.x; it < (nqk + nv) / 8; it += blockDim.x) {
+        float a[8];
+        if (it * 8 >= nqk) {
+            const int i = it * 8 - nqk;
+            unpack8(*reinterpret_cast<const uint4*>(v + t * ld + i), a);
+            st8f(vv + t * nv + i, a);
+            continue;
+        }
+        const int i = it * 8;
+        float b[8], lo[8], bi[8], f[8], w[8];
+        unpack8(*reinterpret_cast<const uint4*>(q + t * ld + i), a); unpack8(*reinterpret_cast<const uint4*>(z + t * ld + i), b);
+        ld8f(bias + i, bi); ld8f(lower + i, lo);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) { a[e] = siluf_(a[e]); forget_gate(b[e] + bi[e], lo[e], f[e], w[e]); }
+        st8f(qq + t * nqk + i, a); st8f(dec + t * nqk + i, f); st8f(kk + t * nqk + i, w);
+    }
+}
+
 // ---------------------------------------------------------------------------------------------------------------------------------
 // router by table: one warp per token
 // ---------------------------------------------------------------------------------------------------------------------------------
@@ -310,6 +351,16 @@ cudaError_t hy_lin_prep(bool f32, const HyLinPrep& p, const void* q, const void*
                               decay_head, dec_head, rope_cos, rope_sin, r)
                : launch_plain(hy_lin_prep_kernel<bf>, dim3(r.T), dim3(128), 0, s, p, (const bf*)q, (const bf*)k, (const bf*)v, ld, qq, kk, vv, dec_channel, 1.0f / tau, decay_head,
                               dec_head, rope_cos, rope_sin, r);
+}
+
+cudaError_t hy_forget_prep(bool f32, int heads, int dim, int vdim, const void* q, const void* z, const void* v, int ld, const float* bias, const float* lower, float* qq, float* kk, float* vv,
+                           float* dec, int T, cudaStream_t s) {
+    if (T <= 0) return cudaSuccess;
+    using bf = __nv_bfloat16;
+    if (heads * dim % 8 == 0 && heads * vdim % 8 == 0 && lin_vec8_ok(f32, 8, 8, 0, ld, q, z, v, qq, kk, vv, dec, bias, lower))      // by the model's sizes alone
+        return launch_plain(hy_forget_prep_vec8_kernel, dim3(T), dim3(128), 0, s, heads * dim, heads * vdim, (const bf*)q, (const bf*)z, (const bf*)v, ld, bias, lower, qq, kk, vv, dec);
+    return f32 ? launch_plain(hy_forget_prep_kernel<float>, dim3(T), dim3(128), 0, s, heads, dim, vdim, (const float*)q, (const float*)z, (const float*)v, ld, bias, lower, qq, kk, vv, dec)
+               : launch_plain(hy_forget_prep_kernel<bf>, dim3(T), dim3(128), 0, s, heads, dim, vdim, (const bf*)q, (const bf*)z, (const bf*)v, ld, bias, lower, qq, kk, vv, dec);
 }
 
 cudaError_t hy_mlstm_gates(const float* gates, int ldg, int heads, float cap, float* mstate, float* dec, float* gin, float* floor_, const HyRows& r, cudaStream_t s) {

@@ -110,6 +110,31 @@ std::vector<float> HybridModel::vec(const std::string& name, int n, float init_m
     }
     return v;
 }
+float* HybridModel::norm_weight(const std::string& name) {
+    std::vector<float> v = vec(name, hc_.width, hc_.norm_around_zero ? 0.f : 1.f, 0.1f);
+    if (hc_.norm_around_zero) for (float& x : v) x += 1.f;
+    return upload_f32(v);
+}
+// The bias table has B rows: distances below B / 2 have a row each, beyond that row B / 2 + floor(ln(n / (B / 2)) / ln(bias_max / (B / 2)) (B - B / 2)),
+// at most B - 1.  Unfolded to one entry per distance up to the first that takes the last row for good; a relative 1e-9 keeps exact powers on
+// their own side of the floor.  run[n]: how far the row of distance n reaches.
+void HybridModel::distance_bias(LayerW& w, const HyLayer& l, const std::string& name) {
+    int B = 32;
+    if (st_) { const StTensor& t = st_->st.get(name); if (t.shape.size() != 2) throw std::runtime_error("checkpoint tensor " + name + " does not have the shape the configuration implies"); B = (int)t.shape[0]; }
+    const std::vector<float> tab = vec(name, B * l.heads, 0.f, 0.5f);
+    const int half = B / 2;
+    if (B < 2 || l.bias_max <= half) throw std::runtime_error("checkpoint tensor " + name + ": bias_max must be more than half of the table's rows");
+    const int L = l.bias_max + 1;
+    std::vector<int32_t> row(L), run(L);
+    for (int n = 0; n < L; ++n)
+        row[n] = n < half ? n : std::min(B - 1, half + (int)std::floor(std::log((double)n / half) / std::log((double)l.bias_max / half) * (B - half) + 1e-9));
+    for (int n = L - 1; n >= 0; --n) run[n] = row[n] == row[L - 1] ? INT32_MAX : row[n] == row[n + 1] ? run[n + 1] : n;
+    std::vector<float> bias((size_t)l.heads * L);
+    for (int h = 0; h < l.heads; ++h) for (int n = 0; n < L; ++n) bias[(size_t)h * L + n] = tab[(size_t)row[n] * l.heads + h];
+    w.rel = upload_f32(bias); w.rel_len = L;
+    w.rel_run = (int32_t*)dmalloc((size_t)L * 4);
+    cuda_check(cudaMemcpy(w.rel_run, run.data(), (size_t)L * 4, cudaMemcpyHostToDevice), "H2D");
+}
 bool HybridModel::has_tensor(const std::string& name) const { return st_ && st_->st.has(name); }
 // cos / sin of position * f_i, f_i = base^(-2 i / dims), angles in double, [max_seq_len, dims / 2].  With YaRN scaling (sc) the frequency is a
 // blend of f_i and f_i / factor along a ramp over i, and both tables carry the amplitude 0.1 ln(factor) + 1.
@@ -159,15 +184,16 @@ HybridModel::HybridModel(const ModelConfig& c, const EngineOptions& o) : ModelBa
     // ---- weights ----
     embed_ = upload_act(tensor("embed", V, W).v);
     head_ = upload_mat(tensor("head", V, W));
-    final_norm_ = upload_f32(vec("final.norm", W, 1.f, 0.1f));
+    final_norm_ = norm_weight("final.norm");
     if (hc_.loop_times > 0 && hc_.loop_reinject) { loop_in_ = upload_mat(tensor("loop.in", W, 2 * W)); loop_step_ = upload_f32(vec("loop.step", hc_.loop_times * W, 0.f, 0.1f)); }
     lw_.resize(hc_.layers.size());
     int max_in = 8, max_p2 = 8, max_conv = 8, max_mix = 8, max_qabs = 8, max_lat = 8, max_qk = 8, max_v = 8, max_dec = 8, max_h = 8, max_act = 8, max_top = 1, max_E = 1, max_ffp = 16, max_lat_heads = 1, max_kv = 0, max_Eattn = 8, max_mix2 = 0, max_gates = 0, max_cq = 0;
     for (size_t li = 0; li < hc_.layers.size(); ++li) {
         const HyLayer& l = hc_.layers[li]; LayerW& w = lw_[li];
         const std::string p = "l" + std::to_string(li) + ".", mx = p + "mix.";
-        w.norm1 = upload_f32(vec(p + "norm1", W, 1.f, 0.1f));
-        if ((hc_.two_norms || hc_.post_norm || hc_.sequential) && (l.moe.present || (hc_.post_norm && has_tensor(p + "norm2")))) w.norm2 = upload_f32(vec(p + "norm2", W, 1.f, 0.1f));
+        w.norm1 = norm_weight(p + "norm1");
+        if ((hc_.two_norms || hc_.post_norm || hc_.sequential) && (l.moe.present || (hc_.post_norm && has_tensor(p + "norm2")))) w.norm2 = norm_weight(p + "norm2");
+        if (hc_.branch_norm) { w.norm1b = norm_weight(p + "norm1b"); if (l.moe.present) w.norm2b = norm_weight(p + "norm2b"); }
         if (hc_.token_shift && (!st_ || has_tensor(p + "shift"))) w.shift = upload_f32(vec(p + "shift", W, 0.5f, 0.5f));
         if (hc_.sequential && hc_.streams > 0) {
             const int n = hc_.streams;
@@ -199,6 +225,8 @@ HybridModel::HybridModel(const ModelConfig& c, const EngineOptions& o) : ModelBa
             if (l.bias) { bias.resize(up8(rows), 0.f); w.in_bias = upload_f32(bias); w.in_bias_act = upload_act(bias); }
             if (l.qk_norm) { w.q_norm = upload_f32(vec(mx + "q.norm", l.dim, 1.f, 0.1f)); w.k_norm = upload_f32(vec(mx + "k.norm", l.dim, 1.f, 0.1f)); }
             if (l.sink) w.sink = upload_f32(vec(mx + "sink", l.heads, 0.f, 1.f));
+            if (l.bias_max > 0) distance_bias(w, l, mx + "rel");
+            if (l.v_first >= 0) w.vmix = vec(mx + "vmix", 1, 0.5f, 0.2f)[0];
             if (l.out_bias) w.o_bias = upload_f32(vec(mx + "o.b", W, 0.f, 0.1f));
             if (l.conv > 0) {          // short convolutions on q | k | v: one weight table over the fused projection's columns (padding columns: zero taps)
                 w.conv_ch = up8(rows);
@@ -241,7 +269,11 @@ HybridModel::HybridModel(const ModelConfig& c, const EngineOptions& o) : ModelBa
                 w.out_w1 = upload_f32(vec(mx + "left.out", W, 1.f, 0.1f)); w.out_w2 = upload_f32(vec(mx + "right.out", W, 1.f, 0.1f));
                 max_mix2 = std::max(max_mix2, l.heads * l.vdim);
             }
-            w.off_q = seg(lx + "q", qk, false); w.off_k = seg(lx + "k", qk, false); w.off_v = seg(lx + "v", vd, false); w.off_g = seg(lx + "g", vd, false);
+            w.off_q = seg(lx + "q", qk, false);
+            if (n.kind == HY_LIN_FORGET_WRITE) {        // [q | f | v]: the forget gate stands where the others keep their keys; no output gate
+                w.off_k = seg(lx + "f", qk, false); w.off_v = seg(lx + "v", vd, false);
+                w.f_bias = upload_f32(vec(lx + "f.b", qk, 1.5f, 1.f)); w.f_lower = upload_f32(vec(lx + "lower", qk, 0.45f, 0.45f));
+            } else { w.off_k = seg(lx + "k", qk, false); w.off_v = seg(lx + "v", vd, false); w.off_g = seg(lx + "g", vd, false); }
             if (n.kind == HY_LIN_CHANNEL_DECAY) {
                 HostMat a1 = tensor(lx + "a1", st_ ? (int)st_->st.get(lx + "a1").shape[0] : std::max(8, W / 16), W);
                 while (rows % 8) { in.v.resize(in.v.size() + W, 0.f); ++rows; }
@@ -266,7 +298,7 @@ HybridModel::HybridModel(const ModelConfig& c, const EngineOptions& o) : ModelBa
             if (two) { bias.resize(up8(rows), 0.f); w.in_bias = upload_f32(bias); w.in_bias_act = upload_act(bias); }
             w.o = upload_mat(tensor(lx + "o", W, vd));
             max_mix = std::max(max_mix, vd); max_qk = std::max(max_qk, qk); max_v = std::max(max_v, vd);
-            max_dec = std::max(max_dec, n.kind == HY_LIN_CHANNEL_DECAY ? qk : n.heads); max_h = std::max(max_h, n.heads);
+            max_dec = std::max(max_dec, n.kind == HY_LIN_CHANNEL_DECAY || n.kind == HY_LIN_FORGET_WRITE ? qk : n.heads); max_h = std::max(max_h, n.heads);
         } else if (l.type == HY_LATENT_ATTENTION) {
             const int qd = l.heads * (l.dim + l.rot_dim), E = l.kv_rank + l.rot_dim;
             if (l.q_rank > 0) {        // queries through a latent: [dq | dkv (| g)] in the fused projection, W_uq as a second stage after the latent's norm
@@ -348,6 +380,7 @@ HybridModel::HybridModel(const ModelConfig& c, const EngineOptions& o) : ModelBa
         if (l.moe.present && l.moe.dense) {
             const std::string mp = p + "mlp.";
             w.up = upload_mat(tensor(mp + "up", l.moe.ff, W)); w.dn = upload_mat(tensor(mp + "down", W, l.moe.ff));
+            if (l.moe.act == HY_EXPERT_POLY_NORM) { const std::vector<float> a = vec(mp + "act", 4, 0.5f, 0.4f); w.poly = HyPolyCoef{a[0], a[1], a[2], a[3]}; }
             max_act = std::max(max_act, up8(l.moe.ff));
         } else if (l.moe.present) {
             const HyMoe& m = l.moe; const std::string mp = p + "mlp.";
@@ -371,7 +404,8 @@ HybridModel::HybridModel(const ModelConfig& c, const EngineOptions& o) : ModelBa
                 if (m.shared_ff > 0) { std::vector<float> sg = tensor(mp + "shared.sg", 1, W).v; sg.resize(Wld_, 0.f); w.shared_gate = upload_act(sg); }
             } else {
             w.router = upload_mat(tensor(mp + "router", m.experts, W));
-            if (m.router == HY_ROUTER_SOFTMAX_CHOSEN) w.router_bias = upload_f32(vec(mp + "router.b", m.experts, 0.f, 0.05f));
+            if (m.router == HY_ROUTER_SIGMOID_CHOSEN) w.router.N = up8(m.experts);      // the padded rows are part of the product: any number of experts fits the tensor-core tile's store
+            else if (m.router == HY_ROUTER_SOFTMAX_CHOSEN) w.router_bias = upload_f32(vec(mp + "router.b", m.experts, 0.f, 0.05f));
             else w.correction = upload_f32(vec(mp + "correction", m.experts, 0.f, 0.05f));
             }
             w.ffp = up16(w.ff_max);
@@ -421,7 +455,7 @@ HybridModel::HybridModel(const ModelConfig& c, const EngineOptions& o) : ModelBa
     dec_ = (float*)dmalloc(MR * max_dec * 4); beta_ = (float*)dmalloc(MR * max_h * 4);
     idx_ = (int32_t*)dmalloc(MR * max_top * 4); wgt_ = (float*)dmalloc(MR * max_top * 4);
     max_tiles_ = (int)((MR * max_top + 127) / 128) + max_E;
-    rlog_ = (float*)dmalloc(MR * max_E * 4);
+    rlog_ = (float*)dmalloc(MR * up8(max_E) * 4);
     bool any_moe_tc = false; for (const LayerW& w : lw_) any_moe_tc |= w.moe_tc;
     act_ = dmalloc(std::max(MR * max_act, any_moe_tc ? (size_t)max_tiles_ * 128 * max_ffp : 0) * es_);
     if (any_moe_tc) {
@@ -529,21 +563,24 @@ void HybridModel::gemm(int mode, const void* A, int lda, const Mat& B, void* C, 
     cuda_check(launch_gemm(&tmA, &B.tm[bn == 32 ? 0 : bn == 64 ? 1 : bn == 128 ? 2 : 3], g, EPI_F32, bn, stream), "gemm (tcgen05, fp32 out)");
 }
 
-void HybridModel::moe(const LayerW& w, const HyLayer& l, const void* h_in, const HyRows& r, const std::function<void(int)>& MARK, const int32_t* tokens, float beta) {
+bool HybridModel::moe(const LayerW& w, const HyLayer& l, const void* h_in, const HyRows& r, const std::function<void(int)>& MARK, const int32_t* tokens, float beta) {
     const HyMoe& m = l.moe; const int W = hc_.width, T = r.T;
+    float* out = x_;
+    if (hc_.sequential) { out = y_; beta = 0.f; }        // the residual is closed by whoever opens the next sublayer
     const bool relu2 = m.act == HY_EXPERT_RELU2; const int rows1 = relu2 ? w.ffp : 2 * w.ffp;
     if (m.dense) {        // one feed-forward for every row: up product with the activation in its epilogue, down product into the sublayer's fp32 output
         gemm(HY_STORE, h_in, Wld_, w.up, act_, up8(m.ff), T, nullptr, 1.f, nullptr, relu2 ? 1 : m.act == HY_EXPERT_GELU_TANH ? 2 : 0); MARK(25);
+        if (m.act == HY_EXPERT_POLY_NORM) { cuda_check(hy_poly_norm(f32_, act_, up8(m.ff), m.ff, w.poly, hc_.eps, T, stream), "poly norm"); MARK(30); }
         gemm(HY_STORE_F32, act_, up8(m.ff), w.dn, y_, W, T, nullptr, 1.f); MARK(26);
-        return;
+        return false;
     }
     HyRouter hr{m.experts, m.top, m.groups, m.keep, m.scale, m.router};
     if (m.router == HY_ROUTER_TOKEN_TABLE) {
         cuda_check(hy_moe_router_table(f32_, tokens, w.table, hc_.vocab, m.top, m.shared_ff > 0 ? m.experts : -1, h_in, Wld_, w.shared_gate, W, idx_, wgt_, T, stream), "router (table)");
     } else {
         // router logits: bf16 (or fp32) inputs, exact products, fp32 accumulation and output
-        gemm(HY_STORE_F32, h_in, Wld_, w.router, rlog_, m.experts, T, nullptr, 1.f);
-        if (m.router == HY_ROUTER_SOFTMAX_CHOSEN) cuda_check(hy_moe_router_softmax(hr, rlog_, m.experts, w.router_bias, idx_, wgt_, T, stream), "router");
+        gemm(HY_STORE_F32, h_in, Wld_, w.router, rlog_, w.router.N, T, nullptr, 1.f);
+        if (m.router == HY_ROUTER_SOFTMAX_CHOSEN || m.router == HY_ROUTER_SIGMOID_CHOSEN) cuda_check(hy_moe_router_softmax(hr, rlog_, w.router.N, w.router_bias, idx_, wgt_, T, stream), "router");
         else cuda_check(hy_moe_router(hr, rlog_, m.experts, w.correction, idx_, wgt_, T, stream), "router");
     }
     MARK(12);
@@ -558,31 +595,36 @@ void HybridModel::moe(const LayerW& w, const HyLayer& l, const void* h_in, const
             make_tmap_bf16_2d(&tmB, act_, (uint64_t)bound * 128, (uint64_t)w.ffp, (uint64_t)w.ffp, 128, 64) != 0) throw std::runtime_error("tensor map for the expert activations failed");
         GemmParams g{}; g.M = bound * 128; g.N = rows1; g.K = Wld_; g.out = act_; g.ldo = w.ffp; g.store_act = relu2 ? 1 : 0;
         g.m_tile_group = tile_expert_; g.n_m_tiles = n_tiles_; g.group_rows = rows1;
+        if (m.act == HY_EXPERT_CLAMPED_GLU) { g.glu_limit = m.limit; g.glu_slope = HY_CLAMPED_GLU_SLOPE; if (m.weight_on_input) { g.row_scale = wgt_; g.row_scale_idx = row_src_; } }
         const int bn1 = rows1 >= 256 ? 256 : 128;
         cuda_check(launch_gemm(&tmA, &w.tm_gu[bn1 == 256], g, relu2 ? EPI_STORE : EPI_SWIGLU, bn1, stream), "experts first stage (grouped tcgen05)"); MARK(17);
         GemmParams d{}; d.M = bound * 128; d.N = W; d.K = w.ffp; d.f32_out = moe_y_; d.ldf = W; d.alpha = 1.f;
         d.m_tile_group = tile_expert_; d.n_m_tiles = n_tiles_; d.group_rows = W;
         const int bn2 = W >= 256 ? 256 : 128;
         cuda_check(launch_gemm(&tmB, &w.tm_down[bn2 == 256], d, EPI_F32, bn2, stream), "experts down (grouped tcgen05)"); MARK(18);
-        cuda_check(hy_moe_combine(moe_y_, W, dst_of_, wgt_, w.n_top, x_, W, T, stream, beta), "expert combine"); MARK(19);
-        return;
+        if (hc_.branch_norm && m.weight_on_input) return true;        // the norm behind the sublayer adds the choices itself
+        cuda_check(hy_moe_combine(moe_y_, W, dst_of_, m.weight_on_input ? nullptr : wgt_, w.n_top, out, W, T, stream, beta), "expert combine"); MARK(19);
+        return false;
     }
-    cuda_check(hy_moe_gate_up(f32_, relu2, h_in, Wld_, w.gu, Wld_, W, w.ff_max, w.ffp, idx_, w.n_top, act_, T, stream), "experts first stage");
-    cuda_check(hy_moe_down(f32_, act_, w.down, W, w.ffp, idx_, wgt_, w.n_top, x_, T, stream, beta), "experts down"); MARK(13);
+    const HyExpertForm form{relu2 ? 1 : m.act == HY_EXPERT_CLAMPED_GLU ? 2 : 0, m.limit, HY_CLAMPED_GLU_SLOPE, m.weight_on_input ? wgt_ : nullptr};
+    cuda_check(hy_moe_gate_up(f32_, form, h_in, Wld_, w.gu, Wld_, W, w.ff_max, w.ffp, idx_, w.n_top, act_, T, stream), "experts first stage");
+    cuda_check(hy_moe_down(f32_, act_, w.down, W, w.ffp, idx_, m.weight_on_input ? nullptr : wgt_, w.n_top, out, T, stream, beta), "experts down"); MARK(13);
+    return false;
 }
 
 const char* HybridModel::kt_name(int id) const {
     static const char* n[32] = {"h2d+embed", "layer_norm", "in_proj_gemm", "latent_absorb+up_gemm", "latent_cache_write", "latent_attention", "conv", "recurrence_prep",
                                 "recurrence", "gated_norm", "low_rank_gemm", "out_proj_gemm", "router", "experts_per_token", "loop_in", "head+argmax",
                                 "expert_plan+gather", "expert_gate_up_gemm", "expert_down_gemm", "expert_combine", "context_gather+kv_up_gemm", "attention_prefill_form", "rms_norm", "window_qk_norm+cache_write",
-                                "window_attention", "dense_ff_up_gemm", "dense_ff_down_gemm", "post_norm", "linear_attention_prep", "memory_gates", "", ""};
+                                "window_attention", "dense_ff_up_gemm", "dense_ff_down_gemm", "post_norm", "linear_attention_prep", "memory_gates", "poly_norm", "branch_norm"};
     return n[id & 31];
 }
 
-static HyWinAttn win_params(const HyLayer& l, float lambda) {
-    HyWinAttn a{l.heads, l.kv_heads, l.dim, l.vdim, l.maps, l.window, l.keep_first, l.qk_norm, l.gate, l.scale, lambda, 1.f - l.diff};
+HyWinAttn HybridModel::window_params(const HyLayer& l, const LayerW& w) const {
+    HyWinAttn a{l.heads, l.kv_heads, l.dim, l.vdim, l.maps, l.window, l.keep_first, l.qk_norm, l.gate, l.scale, w.lambda, 1.f - l.diff};
     a.softcap = l.softcap; a.slope_exp = l.slope_exp; a.q_temp_coef = l.q_temp_coef; a.q_temp_every = l.q_temp_every;
-    a.out_rot = l.v_rot ? (l.rot_layout == HY_ROT_HALVES ? 2 : 1) : 0;
+    if (l.v_rot) { a.out_rot = l.rot_layout == HY_ROT_HALVES ? 2 : 1; a.out_cos = ropes_[w.rope_v].cos; a.out_sin = ropes_[w.rope_v].sin; }
+    a.rel = w.rel; a.rel_run = w.rel_run; a.rel_len = w.rel_len;
     return a;
 }
 
@@ -598,6 +640,10 @@ void HybridModel::linear_mixer(const HyRun& run, const HyLayer& l, const LayerW&
         cuda_check(hy_lin_prep(f32_, HyLinPrep{H, D, VD, n.q_scaled, n.k_scaled, 0}, q, k, v, ld_proj_, qq_, kk_, vv_, dec_, n.tau, nullptr, nullptr, nullptr, nullptr, r, stream), "linear attention operands"); MARK(28);
         cuda_check(hy_recurrence(HY_REC_CHANNEL, qq_, kk_, vv_, dec_, nullptr, rec_, st, H, H, D, VD, r, stream), "gated linear attention"); MARK(8);
         cuda_check(hy_gated_norm(f32_, rec_, H * VD, VD, w.norm_w, VD, g, ld_proj_, 0, n.gate_silu, nullptr, 1, nullptr, 0, mix_, ld_mix_, hc_.eps, T, stream), "gated norm"); MARK(9);
+    } else if (n.kind == HY_LIN_FORGET_WRITE) {
+        cuda_check(hy_forget_prep(f32_, H, D, VD, q, k, v, ld_proj_, w.f_bias, w.f_lower, qq_, kk_, vv_, dec_, T, stream), "forget gate operands"); MARK(28);
+        cuda_check(hy_recurrence(HY_REC_CHANNEL, qq_, kk_, vv_, dec_, nullptr, rec_, st, H, H, D, VD, r, stream), "forget-gate recurrence"); MARK(8);
+        cuda_check(hy_gated_norm(f32_, rec_, H * VD, VD, w.norm_w, VD, nullptr, 4, 0, 0, nullptr, 1, nullptr, 0, mix_, ld_mix_, hc_.eps, T, stream), "head norm"); MARK(9);
     } else if (n.kind == HY_LIN_HEAD_DECAY) {
         const float* rc = w.rope >= 0 ? ropes_[w.rope].cos : nullptr; const float* rs = w.rope >= 0 ? ropes_[w.rope].sin : nullptr;
         cuda_check(hy_lin_prep(f32_, HyLinPrep{H, D, VD, n.q_scaled, n.k_scaled, n.rot_dims}, q, k, v, ld_proj_, qq_, kk_, vv_, nullptr, 1.f, w.decay, dec_, rc, rs, r, stream), "retention operands"); MARK(28);
@@ -622,9 +668,16 @@ HyLatentAttn HybridModel::latent_params(const HyLayer& l, const LayerW& w) const
 
 void HybridModel::window_mixer(const HyRun& run, const HyLayer& l, const LayerW& w, const HyRows& r, const TileList& tl, const std::function<void(int)>& MARK, void* q, void* k, void* v, int ld,
                                const void* gate, int ldg, bool prepared) {
-    HyWinAttn a{l.heads, l.kv_heads, l.dim, l.vdim, l.maps, l.window, l.keep_first, l.qk_norm, l.gate, l.scale, w.lambda, 1.f - l.diff};
-    if (l.v_rot) { a.out_rot = l.rot_layout == HY_ROT_HALVES ? 2 : 1; a.out_cos = ropes_[w.rope_v].cos; a.out_sin = ropes_[w.rope_v].sin; }
-    if (!prepared && (l.rot_dims > 0 || l.v_rot)) {
+    const HyWinAttn a = window_params(l, w);
+    if (!prepared && l.v_norm) {
+        HyValueMix vm{nullptr, 0, 0, w.vmix};
+        if (l.v_first >= 0) {       // the first mixing layer has cached this token's value earlier in the same step
+            const HyLayer& f = hc_.layers[l.v_first];
+            for (const HyRun& o : hc_.runs) if (o.layer == l.v_first) vm.first = caches_[o.cache_idx];
+            vm.first_row = cache_row_width(f); vm.first_col = f.kv_heads * f.maps * f.dim;
+        }
+        cuda_check(hy_win_value_prep(f32_, a, k, v, ld, vm, hc_.eps, caches_[run.cache_idx], r, stream), "value norm + cache write");
+    } else if (!prepared && (l.rot_dims > 0 || l.v_rot)) {
         const HyRotary rot{l.rot_dims, l.rot_layout, l.rot_dims > 0 ? ropes_[w.rope].cos : nullptr, l.rot_dims > 0 ? ropes_[w.rope].sin : nullptr,
                            l.v_rot ? ropes_[w.rope_v].cos : nullptr, l.v_rot ? ropes_[w.rope_v].sin : nullptr};
         cuda_check(hy_win_rope_prep(f32_, a, rot, q, ld, k, v, ld, caches_[run.cache_idx], r, stream), "rotary + cache write");
@@ -683,7 +736,13 @@ void HybridModel::forward_sequential(const HyRows& r, const std::vector<TileList
     const bool hyper = hc_.streams > 0;
     const float *pend_mix = nullptr, *pend_out = nullptr;      // coefficients of the sublayer whose y_ has not been folded into the streams yet
     bool pending = false;
+    HyBranch branch{nullptr, nullptr, hc_.residual_mult, nullptr, 0};        // designs with a norm behind the sublayer: the one that has not joined the residual yet
     auto open = [&](const float* in, const float* norm_w, float* shift_state, const char* what) {
+        if (hc_.branch_norm) {
+            cuda_check(hy_branch_norm(f32_, xs_, branch, nullptr, norm_w, hc_.eps, h_, Wld_, T, W, stream), what);
+            branch.y = nullptr;
+            return;
+        }
         const HyStreams c{n, pend_mix, pend_out, in};
         cuda_check(hy_stream_norm(f32_, c, xs_, pending ? y_ : nullptr, nullptr, norm_w, hc_.eps, h_, Wld_, hn_, shift_state, shift_prev_, r, T, W, stream), what);
         pending = false;
@@ -693,9 +752,10 @@ void HybridModel::forward_sequential(const HyRows& r, const std::vector<TileList
         float* sstate = w.shift ? shift_states_[run.index] : nullptr;
         open(hyper ? w.hc_in[0] : ones_, w.norm1, sstate, "streams + norm (mixer)");
         if (sstate) cuda_check(hy_token_shift(f32_, hn_, shift_prev_, w.shift, h_, Wld_, r, W, stream), "token shift");
-        MARK(22);
+        MARK(hc_.branch_norm ? 31 : 22);
         gemm(HY_STORE, h_, Wld_, w.in, proj_, ld_proj_, T, w.in_bias, 1.f, w.in_bias_act); MARK(2);
-        if (l.type == HY_LATENT_ATTENTION) {
+        if (l.type == HY_LINEAR_ATTENTION) linear_mixer(run, l, w, r, MARK);
+        else if (l.type == HY_LATENT_ATTENTION) {
             void* q = at(proj_, w.off_a); int ldq = ld_proj_;
             if (l.q_rank > 0) {
                 cuda_check(hy_rmsnorm_act(f32_, at(proj_, w.off_a), ld_proj_, l.q_rank, w.dq_norm, cq_, ld_cq_, hc_.eps, T, stream), "query latent norm");
@@ -705,7 +765,7 @@ void HybridModel::forward_sequential(const HyRows& r, const std::vector<TileList
             latent_mixer(run, l, w, r, tile_lists[run.layer], MARK, q, ldq, at(proj_, w.off_b), ld_proj_, l.gate == HY_GATE_CHANNEL ? at(proj_, w.off_d) : nullptr, ld_proj_);
         } else if (l.type == HY_WINDOW_ATTENTION) {
             void* src = proj_; int ld = ld_proj_;
-            const HyWinAttn wa = win_params(l, 0.f);
+            const HyWinAttn wa = window_params(l, w);
             const HyRotary rot{l.rot_dims, l.rot_layout, l.rot_dims > 0 ? ropes_[w.rope].cos : nullptr, l.rot_dims > 0 ? ropes_[w.rope].sin : nullptr,
                                l.v_rot ? ropes_[w.rope_v].cos : nullptr, l.v_rot ? ropes_[w.rope_v].sin : nullptr};
             if (!f32_ && l.conv > 1 && run.cache_owner && hy_conv_rope_cache_supported(wa, rot, l.conv)) {
@@ -725,9 +785,11 @@ void HybridModel::forward_sequential(const HyRows& r, const std::vector<TileList
         } else throw std::runtime_error("forward: this design has no such mixer");
         gemm(HY_STORE_F32, mix_, ld_mix_, w.o, y_, W, T, w.o_bias, 1.f); MARK(11);
         pending = true; pend_mix = hyper ? w.hc_mix[0] : ones_; pend_out = hyper ? w.hc_out[0] : ones_;
+        branch.y = y_; branch.w = w.norm1b; branch.dst_of = nullptr;
         if (l.moe.present) {
-            open(hyper ? w.hc_in[1] : ones_, w.norm2, nullptr, "streams + norm (feed-forward)"); MARK(22);
-            moe(w, l, h_, r, MARK, d_tokens);
+            open(hyper ? w.hc_in[1] : ones_, w.norm2, nullptr, "streams + norm (feed-forward)"); MARK(hc_.branch_norm ? 31 : 22);
+            const bool spread = moe(w, l, h_, r, MARK, d_tokens);
+            branch.y = spread ? moe_y_ : y_; branch.w = w.norm2b; branch.dst_of = spread ? dst_of_ : nullptr; branch.top = w.n_top;
             pending = true; pend_mix = hyper ? w.hc_mix[1] : ones_; pend_out = hyper ? w.hc_out[1] : ones_;
         }
         if (capture_layers) {          // debug: the residual (sum of the streams) after this execution
@@ -739,6 +801,7 @@ void HybridModel::forward_sequential(const HyRows& r, const std::vector<TileList
             for (int t = 0; t < T; ++t) for (int sidx = 0; sidx < n; ++sidx) for (int c = 0; c < W; ++c) (*capture_layers)[n0 + (size_t)t * W + c] += tmp[((size_t)t * n + sidx) * W + c];
         }
     }
+    pend_branch_ = branch;
     pending_ = pending; pend_mix_ = pend_mix; pend_out_ = pend_out;      // the final norm folds the last y_ into the rows it reads; the streams themselves are not needed again
 }
 
@@ -773,7 +836,7 @@ void HybridModel::forward(const StepInput& in, float* logits_out) {
         const HyLayer& l = hc_.layers[li]; TileList& tl = tile_lists[li];
         if (l.type == HY_WINDOW_ATTENTION || l.type == HY_ATTENTION_BESIDE_MEMORY) {
             // windowed attention on the tensor cores: tiles of 64 consecutive (row, head-of-the-group) pairs of one sequence; a decoding row is one tile per key/value head
-            tl.mma = !f32_ && opt.hy_tensor_core && ld_proj_ % 8 == 0 && (l.type == HY_WINDOW_ATTENTION ? ld_mix_ : ld_mix2_) % 8 == 0 && hy_win_mma_supported(win_params(l, 0.f));
+            tl.mma = !f32_ && opt.hy_tensor_core && ld_proj_ % 8 == 0 && (l.type == HY_WINDOW_ATTENTION ? ld_mix_ : ld_mix2_) % 8 == 0 && hy_win_mma_supported(window_params(l, lw_[li]));
             if (!tl.mma) continue;
             tile_seq_.clear(); tile_q0_.clear(); ptile_seq_.clear(); ptile_row0_.clear();
             const int group = l.heads / l.kv_heads;
@@ -858,7 +921,7 @@ void HybridModel::forward(const StepInput& in, float* logits_out) {
             gemm(HY_STORE, h_, Wld_, w.in, proj_, ld_proj_, T, w.in_bias, 1.f, w.in_bias_act); MARK(2);
             const bool two = l.type == HY_ATTENTION_BESIDE_MEMORY;
             if (two) {
-                const HyWinAttn a = win_params(l, 0.f);
+                const HyWinAttn a = window_params(l, w);
                 cuda_check(hy_win_prep(f32_, a, at(proj_, w.off_lq), ld_proj_, at(proj_, w.off_lk), at(proj_, w.off_lv), ld_proj_, w.q_norm, w.k_norm, hc_.eps, caches_[run.cache_idx], r, stream),
                            "query / key norm + cache write"); MARK(23);
                 const TileList& tl = tile_lists[run.layer];
@@ -931,7 +994,9 @@ void HybridModel::forward(const StepInput& in, float* logits_out) {
         capture_layers = nullptr;
     }
     if (NS > 0) {
-        if (hc_.sequential) {      // x = the sum of the streams, of the wanted rows only
+        if (hc_.branch_norm) {
+            cuda_check(hy_branch_norm(f32_, xs_, pend_branch_, d_meta_ + o_samp, final_norm_, hc_.eps, hs_, Wld_, NS, W, stream), "final norm");
+        } else if (hc_.sequential) {      // x = the sum of the streams, of the wanted rows only
             const HyStreams fin{n_streams_, pend_mix_, pend_out_, ones_};
             cuda_check(hy_stream_norm(f32_, fin, xs_, pending_ ? y_ : nullptr, d_meta_ + o_samp, final_norm_, hc_.eps, hs_, Wld_, nullptr, nullptr, nullptr, r, NS, W, stream), "final norm");
         } else if (hc_.norm == HY_RMS_NORM) cuda_check(hy_rmsnorm_pair(f32_, x_, d_meta_ + o_samp, final_norm_, hs_, nullptr, nullptr, Wld_, NS, W, hc_.eps, stream), "final norm");

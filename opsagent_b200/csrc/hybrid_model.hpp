@@ -4,7 +4,8 @@
 // 64-token pages, recurrent layers keep an fp32 state and their convolution tails (or, for a matrix memory, its normaliser and running
 // maximum) in the sequence's state slot.  Designs whose norm follows the sum (x <- norm(alpha x + sublayer(x))) run mixer and feed-forward in
 // sequence; pre-norm designs run them either side by side on norms of the same residual or in sequence, the latter optionally on several
-// residual streams (hyper-connections) and with a token shift in front of the mixer whose carried row lives in the state slot too.
+// residual streams (hyper-connections) and with a token shift in front of the mixer whose carried row lives in the state slot too, or with a
+// second norm behind every sublayer.
 #pragma once
 #include <functional>
 #include <string>
@@ -50,6 +51,9 @@ private:
         Mat up, dn;                                   // dense feed-forward
         // designs with sublayers in sequence: token shift weight, hyper-connection coefficients of the mixer (1) and the feed-forward (2), all fp32 on the device
         float *shift = nullptr, *hc_in[2] = {nullptr, nullptr}, *hc_mix[2] = {nullptr, nullptr}, *hc_out[2] = {nullptr, nullptr}, *o_bias = nullptr;
+        float *norm1b = nullptr, *norm2b = nullptr;    // norms behind the mixer and the feed-forward
+        float* rel = nullptr; int32_t* rel_run = nullptr; int rel_len = 0; float vmix = 0.f;      // bias per (head, distance), see HyWinAttn; share of the first layer's values
+        float *f_bias = nullptr, *f_lower = nullptr; HyPolyCoef poly{0.f, 0.f, 0.f, 0.f};         // forget gate; PolyNorm coefficients
         Mat uq; float* dq_norm = nullptr; int rope_v = -1;      // latent attention with a low-rank query; rotary table of rotated values
         // linear attention and attention beside a matrix memory: segments of the fused input projection, second stage and biases
         int off_q = 0, off_k = 0, off_v = 0, off_g = 0, off_a1 = 0, off_lq = 0, off_lk = 0, off_lv = 0;
@@ -68,9 +72,12 @@ private:
     Mat upload_mat(const HostMat& m);
     HostMat tensor(const std::string& name, int N, int K);                // checkpoint tensor (or seeded values) as fp32 [N, K]; K == 0: any width
     std::vector<float> vec(const std::string& name, int n, float init_mean, float init_spread);
+    float* norm_weight(const std::string& name);                          // [width] weight of a layer norm or the final norm as it multiplies (stored around one or around zero)
+    void distance_bias(LayerW& w, const HyLayer& l, const std::string& name);      // bias table [rows, heads] -> one entry per distance
     void gemm(int mode, const void* A, int lda, const Mat& B, void* C, int ldc, int M, const float* bias, float alpha, const void* bias_act = nullptr, int act = 0);
-    // routed experts (and a dense feed-forward): x = beta x + sum of the chosen experts' outputs
-    void moe(const LayerW& w, const HyLayer& l, const void* h, const HyRows& r, const std::function<void(int)>& mark, const int32_t* tokens = nullptr, float beta = 1.f);
+    // routed experts (and a dense feed-forward): x = beta x + sum of the chosen experts' outputs (sequential designs: the sum alone goes to y_).
+    // Returns true where the caller is to add the choices itself: their rows lie in moe_y_ at dst_of_ (designs with a norm behind the sublayer)
+    bool moe(const LayerW& w, const HyLayer& l, const void* h, const HyRows& r, const std::function<void(int)>& mark, const int32_t* tokens = nullptr, float beta = 1.f);
     int rope_table(float base, int dims, const HyRotScaling* sc = nullptr);
     // latent attention of one layer execution: q [T, ldq] (head by head [dim | rot_dim]) and the down projection ckv [T, ldc] -> heads' outputs in mix_
     void latent_mixer(const HyRun& run, const HyLayer& l, const LayerW& w, const HyRows& r, const TileList& tl, const std::function<void(int)>& mark, void* q, int ldq, void* ckv, int ldc,
@@ -79,6 +86,7 @@ private:
     void window_mixer(const HyRun& run, const HyLayer& l, const LayerW& w, const HyRows& r, const TileList& tl, const std::function<void(int)>& mark, void* q, void* k, void* v, int ld,
                       const void* gate, int ldg, bool prepared = false);      // prepared: queries are rotated and the cache row is written already
     void forward_sequential(const HyRows& r, const std::vector<TileList>& tile_lists, const int32_t* d_tokens, const std::function<void(int)>& mark);
+    HyWinAttn window_params(const HyLayer& l, const LayerW& w) const;
     HyLatentAttn latent_params(const HyLayer& l, const LayerW& w) const;
     void linear_mixer(const HyRun& run, const HyLayer& l, const LayerW& w, const HyRows& r, const std::function<void(int)>& mark);
     bool has_tensor(const std::string& name) const;
@@ -92,6 +100,7 @@ private:
     std::vector<void*> caches_;                    // per attention execution: [num_pages * 64][kv_rank + rot_dim] in the activation type
     std::vector<float*> states_; std::vector<void*> tails_;      // per recurrent execution: [slots][heads * dim * vdim] fp32, [slots][(taps - 1) * channels]
     std::vector<float*> shift_states_;             // per layer execution of a design with a token shift: [slots][width] fp32, the last normed row of the sequence
+    HyBranch pend_branch_{nullptr, nullptr, 0.f, nullptr, 0};      // the same of a design with norms behind its sublayers
     const float *pend_mix_ = nullptr, *pend_out_ = nullptr; bool pending_ = false;      // the last sublayer's y_ is folded into the streams by whoever reads them next
     float *xs_ = nullptr, *hn_ = nullptr, *shift_prev_ = nullptr, *ones_ = nullptr; void* cq_ = nullptr; int ld_cq_ = 0, n_streams_ = 1;      // residual streams [T, n, W]; normed rows before the shift; carried rows of the step's sequences
     std::vector<float*> aux_;                      // per matrix-memory execution: [slots][heads * dim] normaliser, then [slots][heads] running maximum

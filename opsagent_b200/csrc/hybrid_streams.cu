@@ -1,4 +1,4 @@
-// hybrid_streams.cu — the residual of designs whose sublayers run in sequence on several residual streams (API: hybrid_kernels.hpp).
+// hybrid_streams.cu — the residual of designs whose sublayers run in sequence, on several residual streams or on one (API: hybrid_kernels.hpp).
 //
 // Hyper-connections: a row carries n streams x_1..x_n (fp32, [T, n, W]).  A sublayer reads u = sum_s in[s] x_s through its RMS norm and, when
 // it has produced y, every stream becomes x_t <- sum_s mix[s, t] x_s + out[t] y — all from the old streams.  hy_stream_norm does the closing
@@ -9,6 +9,10 @@
 // leaves v in fp32 and hy_token_shift reads rows t and t - 1; across steps the last v of a sequence lives in its state slot.  The exchange
 // with the slot (old row out to `prev`, new row in) is done by the CTA of the sequence's last row, channel by channel by the same thread,
 // so no other CTA reads the slot while it changes.
+//
+// Norms on both sides of a sublayer (one stream): x <- x + m norm_b(y), then h = norm(x) for the next sublayer.  hy_branch_norm does both in one
+// pass with the row in registers; a routed feed-forward's y may still lie in its experts' sorted tiles, the kernel then gathers and adds the
+// token's choices itself.  PolyNorm, the dense activation that needs the whole row (three RMS norms over the width), stands here too.
 #include "hybrid_common.cuh"
 #include "hybrid_kernels.hpp"
 
@@ -177,7 +181,168 @@ cudaError_t stream_norm_t(const HyStreams& c, float* xs, const float* y, const i
     }
 }
 
+// y of one row at channels c .. c + V: the row itself, or the sum of the token's choices in choice order
+template <int V>
+__device__ __forceinline__ void branch_load(const HyBranch& b, long long src, int W, int c, FVec<V>& y) {
+    if (!b.dst_of) { y.load(b.y + src * W + c); return; }
+    y.load(b.y + (long long)b.dst_of[src * b.top] * W + c);
+    for (int k = 1; k < b.top; ++k) {
+        FVec<V> u; u.load(b.y + (long long)b.dst_of[src * b.top + k] * W + c);
+#pragma unroll
+        for (int e = 0; e < V; ++e) y.v[e] += u.v[e];
+    }
+}
+template <typename TA, int NV>      // NV float4 per thread: W <= 1024 NV
+__global__ void __launch_bounds__(256) hy_branch_norm_reg_kernel(float* __restrict__ x, HyBranch b, const int32_t* __restrict__ rows, const float* __restrict__ w, float eps,
+                                                                 TA* __restrict__ h, int ldh, int W) {
+    HY_PDL();
+    __shared__ float red[32];
+    const long long t = blockIdx.x, src = rows ? rows[t] : t;
+    float* xr = x + src * W;
+    FVec<4> v[NV];
+#pragma unroll
+    for (int k = 0; k < NV; ++k) { const int c = (threadIdx.x + k * 256) * 4; if (c < W) v[k].load(xr + c); }
+    if (b.y) {
+        FVec<4> y[NV]; float ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            const int c = (threadIdx.x + k * 256) * 4;
+            if (c < W) { branch_load<4>(b, src, W, c, y[k]); ss += (y[k].v[0] * y[k].v[0] + y[k].v[1] * y[k].v[1]) + (y[k].v[2] * y[k].v[2] + y[k].v[3] * y[k].v[3]); }
+        }
+        const float ry = b.mult / sqrtf(block_sum(ss, red) / (float)W + eps);
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            const int c = (threadIdx.x + k * 256) * 4;
+            if (c < W) {
+                FVec<4> g; g.load(b.w + c);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) v[k].v[e] = fmaf(y[k].v[e] * ry, g.v[e], v[k].v[e]);
+                if (!rows) v[k].store(xr + c);
+            }
+        }
+    }
+    if (!w) return;
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NV; ++k) if ((threadIdx.x + k * 256) * 4 < W) ss += (v[k].v[0] * v[k].v[0] + v[k].v[1] * v[k].v[1]) + (v[k].v[2] * v[k].v[2] + v[k].v[3] * v[k].v[3]);
+    const float rr = 1.0f / sqrtf(block_sum(ss, red) / (float)W + eps);
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int c = (threadIdx.x + k * 256) * 4;
+        if (c < W) {
+            FVec<4> g; g.load(w + c); float o[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) o[e] = v[k].v[e] * rr * g.v[e];
+            store_act<4>(h + t * ldh + c, o);
+        }
+    }
+}
+// any width: what the registers above hold is read again
+template <typename TA>
+__global__ void __launch_bounds__(256) hy_branch_norm_kernel(float* __restrict__ x, HyBranch b, const int32_t* __restrict__ rows, const float* __restrict__ w, float eps,
+                                                             TA* __restrict__ h, int ldh, int W) {
+    HY_PDL();
+    __shared__ float red[32];
+    const long long t = blockIdx.x, src = rows ? rows[t] : t;
+    float* xr = x + src * W;
+    float ry = 0.f;
+    if (b.y) {
+        float ss = 0.f;
+        for (int c = threadIdx.x; c < W; c += blockDim.x) { FVec<1> y; branch_load<1>(b, src, W, c, y); ss = fmaf(y.v[0], y.v[0], ss); }
+        ry = b.mult / sqrtf(block_sum(ss, red) / (float)W + eps);
+    }
+    auto value = [&](int c) { if (!b.y) return xr[c]; FVec<1> y; branch_load<1>(b, src, W, c, y); return fmaf(y.v[0] * ry, b.w[c], xr[c]); };
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < W; c += blockDim.x) {
+        const float v = value(c);
+        ss = fmaf(v, v, ss);
+        if (!rows && b.y) xr[c] = v;                 // a thread reads again only what it alone has written
+    }
+    if (!w) return;
+    const float rr = 1.0f / sqrtf(block_sum(ss, red) / (float)W + eps);
+    for (int c = threadIdx.x; c < W; c += blockDim.x) stf(h + t * ldh + c, (rows ? value(c) : xr[c]) * rr * w[c]);
+}
+
+__device__ __forceinline__ float3 block_sum3(float3 s, float (*red)[32]) {      // three sums over a block of 256 threads at once
+    s.x = warp_sum(s.x); s.y = warp_sum(s.y); s.z = warp_sum(s.z);
+    const int w = threadIdx.x >> 5;
+    if ((threadIdx.x & 31) == 0) { red[0][w] = s.x; red[1][w] = s.y; red[2][w] = s.z; }
+    __syncthreads();
+    float3 t = make_float3(0.f, 0.f, 0.f);
+    for (int i = 0; i < (int)(blockDim.x >> 5); ++i) { t.x += red[0][i]; t.y += red[1][i]; t.z += red[2][i]; }
+    return t;
+}
+struct PolyScale { float a, b, c, e; };
+__device__ __forceinline__ PolyScale poly_scale(const HyPolyCoef& k, float3 s, int n, float eps) {
+    const float m = 1.0f / (float)n;
+    return PolyScale{k.a / sqrtf(s.x * m + eps), k.b / sqrtf(s.y * m + eps), k.c / sqrtf(s.z * m + eps), k.e};
+}
+__device__ __forceinline__ void poly_add(float3& s, float z) { const float z2 = z * z, z3 = z2 * z; s.x += z2; s.y = fmaf(z2, z2, s.y); s.z = fmaf(z3, z3, s.z); }
+__device__ __forceinline__ float poly_value(const PolyScale& p, float z) { return fmaf(z, fmaf(z, fmaf(z, p.c, p.b), p.a), p.e); }      // one polynomial once the three norms are known
+template <typename TA>
+__global__ void __launch_bounds__(256) hy_poly_norm_kernel(TA* __restrict__ z, int ldz, int n, HyPolyCoef k, float eps) {
+    HY_PDL();
+    __shared__ float red[3][32];
+    TA* zr = z + (long long)blockIdx.x * ldz;
+    float3 s = make_float3(0.f, 0.f, 0.f);
+    for (int c = threadIdx.x; c < n; c += blockDim.x) poly_add(s, ldf(zr + c));
+    const PolyScale p = poly_scale(k, block_sum3(s, red), n, eps);
+    for (int c = threadIdx.x; c < n; c += blockDim.x) stf(zr + c, poly_value(p, ldf(zr + c)));
+}
+template <int NV>      // bf16 rows in aligned groups of 8 channels, the row in registers: n <= 2048 NV
+__global__ void __launch_bounds__(256) hy_poly_norm_vec8_kernel(bf* __restrict__ z, int ldz, int n, HyPolyCoef k, float eps) {
+    HY_PDL();
+    __shared__ float red[3][32];
+    bf* zr = z + (long long)blockIdx.x * ldz;
+    uint4 u[NV];
+    float3 s = make_float3(0.f, 0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) { const int c = (threadIdx.x + i * 256) * 8; u[i] = c < n ? *reinterpret_cast<const uint4*>(zr + c) : make_uint4(0, 0, 0, 0); }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const uint32_t x[4] = {u[i].x, u[i].y, u[i].z, u[i].w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) { poly_add(s, bf16lo(x[e])); poly_add(s, bf16hi(x[e])); }
+    }
+    const PolyScale p = poly_scale(k, block_sum3(s, red), n, eps);
+    auto two = [&](uint32_t x) { return pack_bf16x2(poly_value(p, bf16lo(x)), poly_value(p, bf16hi(x))); };
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int c = (threadIdx.x + i * 256) * 8;
+        if (c < n) *reinterpret_cast<uint4*>(zr + c) = make_uint4(two(u[i].x), two(u[i].y), two(u[i].z), two(u[i].w));
+    }
+}
+
+template <typename TA>
+cudaError_t branch_norm_t(float* x, const HyBranch& b, const int32_t* rows, const float* w, float eps, void* h, int ldh, int T, int W, cudaStream_t s) {
+    auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    // the form follows from the model's sizes alone, so a row takes the same kernel in every step
+    if (W % 4 == 0 && W <= 8192 && ldh % 4 == 0 && al16(x) && al16(b.y) && al16(b.w) && al16(w) && al16(h)) {
+        if (W <= 1024) return launch_plain(hy_branch_norm_reg_kernel<TA, 1>, dim3(T), dim3(256), 0, s, x, b, rows, w, eps, (TA*)h, ldh, W);
+        if (W <= 2048) return launch_plain(hy_branch_norm_reg_kernel<TA, 2>, dim3(T), dim3(256), 0, s, x, b, rows, w, eps, (TA*)h, ldh, W);
+        if (W <= 4096) return launch_plain(hy_branch_norm_reg_kernel<TA, 4>, dim3(T), dim3(256), 0, s, x, b, rows, w, eps, (TA*)h, ldh, W);
+        return launch_plain(hy_branch_norm_reg_kernel<TA, 8>, dim3(T), dim3(256), 0, s, x, b, rows, w, eps, (TA*)h, ldh, W);
+    }
+    return launch_plain(hy_branch_norm_kernel<TA>, dim3(T), dim3(256), 0, s, x, b, rows, w, eps, (TA*)h, ldh, W);
+}
+
 }  // namespace
+
+cudaError_t hy_branch_norm(bool f32, float* x, const HyBranch& b, const int32_t* rows, const float* w, float eps, void* h, int ldh, int T, int W, cudaStream_t s) {
+    if (T <= 0) return cudaSuccess;
+    return f32 ? branch_norm_t<float>(x, b, rows, w, eps, h, ldh, T, W, s) : branch_norm_t<bf>(x, b, rows, w, eps, h, ldh, T, W, s);
+}
+cudaError_t hy_poly_norm(bool f32, void* z, int ldz, int n, const HyPolyCoef& k, float eps, int T, cudaStream_t s) {
+    if (T <= 0) return cudaSuccess;
+    if (f32) return launch_plain(hy_poly_norm_kernel<float>, dim3(T), dim3(256), 0, s, (float*)z, ldz, n, k, eps);
+    if (n % 8 == 0 && ldz % 8 == 0 && (reinterpret_cast<uintptr_t>(z) & 15) == 0 && n <= 16384) {
+        if (n <= 2048) return launch_plain(hy_poly_norm_vec8_kernel<1>, dim3(T), dim3(256), 0, s, (bf*)z, ldz, n, k, eps);
+        if (n <= 4096) return launch_plain(hy_poly_norm_vec8_kernel<2>, dim3(T), dim3(256), 0, s, (bf*)z, ldz, n, k, eps);
+        if (n <= 8192) return launch_plain(hy_poly_norm_vec8_kernel<4>, dim3(T), dim3(256), 0, s, (bf*)z, ldz, n, k, eps);
+        return launch_plain(hy_poly_norm_vec8_kernel<8>, dim3(T), dim3(256), 0, s, (bf*)z, ldz, n, k, eps);
+    }
+    return launch_plain(hy_poly_norm_kernel<bf>, dim3(T), dim3(256), 0, s, (bf*)z, ldz, n, k, eps);
+}
 
 cudaError_t hy_embed_streams(bool f32, const int32_t* ids, const void* table, float* xs, int T, int W, int vocab, float scale, int n, cudaStream_t s) {
     return f32 ? launch_plain(hy_embed_streams_kernel<float>, dim3(T), dim3(256), 0, s, ids, (const float*)table, xs, W, vocab, scale, n)

@@ -7,7 +7,8 @@
 // sequence; an optional RMS norm of every query / key map; an optional sink logit per head that only enlarges the softmax denominator; a
 // sigmoid output gate per channel or per head; optional score modifiers — a soft cap (cap tanh(score / cap)) and a penalty per position of
 // distance with a slope per head — and, in the preparation step, one RMS norm over the whole query / key projection and a query temperature
-// that grows with the logarithm of the position.  Softmax, norms, score modifiers and gates are fp32 in both element types.
+// that grows with the logarithm of the position, or a learned bias per head and distance (a table over distances; the query temperature then
+// multiplies the scores) with values cached at unit RMS and mixed with another layer's.  Softmax, norms, score modifiers and gates are fp32 in both element types.
 #include "hybrid_common.cuh"
 #include "hybrid_kernels.hpp"
 
@@ -276,6 +277,54 @@ __global__ void __launch_bounds__(128) hy_conv_rope_cache_kernel(HyWinAttn a, Hy
     }
 }
 
+// Preparation of a layer with unit-RMS values: per row, keys are copied into the row's cache slot, every value head is divided by its RMS and, where a
+// first layer is given, mixed with that layer's cached value of the same token.  One warp per value head, the copy spread over the CTA.
+template <typename TA>
+__global__ void __launch_bounds__(128) hy_win_value_prep_kernel(HyWinAttn a, const TA* __restrict__ k, const TA* __restrict__ v, int ldkv, const TA* __restrict__ first, int first_row,
+                                                                int first_col, float lambda, float eps, TA* __restrict__ cache, HyRows r) {
+    HY_PDL();
+    const long long t = blockIdx.x, slot = r.slots[t]; const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, VD = a.vdim;
+    const int KW = a.kv_heads * a.dim, CW = KW + a.kv_heads * VD;
+    TA* crow = cache + slot * CW;
+    for (int c = threadIdx.x; c < KW; c += blockDim.x) crow[c] = k[t * ldkv + c];
+    for (int g = warp; g < a.kv_heads; g += 4) {
+        const TA* src = v + t * ldkv + (long long)g * VD; const TA* fr = first ? first + slot * first_row + first_col + (long long)g * VD : nullptr;
+        float ss = 0.f;
+        for (int c = lane; c < VD; c += 32) { const float x = ldf(src + c); ss = fmaf(x, x, ss); }
+        const float rr = 1.0f / sqrtf(warp_sum(ss) / (float)VD + eps);
+        for (int c = lane; c < VD; c += 32) {
+            float x = ldf(src + c) * rr;
+            if (fr) x = (1.0f - lambda) * x + lambda * ldf(fr + c);
+            stf(crow + KW + (long long)g * VD + c, x);
+        }
+    }
+}
+// bf16 rows in aligned groups of 8 channels with vdim / 8 a power of two up to 32 lanes: 16 bytes per access, the lanes of a value head meet by shuffles
+__global__ void __launch_bounds__(128) hy_win_value_prep_vec8_kernel(HyWinAttn a, const __nv_bfloat16* __restrict__ k, const __nv_bfloat16* __restrict__ v, int ldkv,
+                                                                     const __nv_bfloat16* __restrict__ first, int first_row, int first_col, float lambda, float eps,
+                                                                     __nv_bfloat16* __restrict__ cache, HyRows r) {
+    HY_PDL();
+    const long long t = blockIdx.x, slot = r.slots[t]; const int tid = threadIdx.x, GS = a.vdim / 8;
+    const int KW = a.kv_heads * a.dim, VW = a.kv_heads * a.vdim, CW = KW + VW;
+    __nv_bfloat16* crow = cache + slot * CW;
+    for (int base = 0; base < VW; base += 128 * 8) {
+        const int c = base + tid * 8; const bool ok = c < VW;
+        uint4 raw = make_uint4(0, 0, 0, 0), fr = make_uint4(0, 0, 0, 0);
+        if (ok) { raw = *reinterpret_cast<const uint4*>(v + t * ldkv + c); if (first) fr = *reinterpret_cast<const uint4*>(first + slot * first_row + first_col + c); }
+        const float x[8] = {bf16lo(raw.x), bf16hi(raw.x), bf16lo(raw.y), bf16hi(raw.y), bf16lo(raw.z), bf16hi(raw.z), bf16lo(raw.w), bf16hi(raw.w)};
+        const float f[8] = {bf16lo(fr.x), bf16hi(fr.x), bf16lo(fr.y), bf16hi(fr.y), bf16lo(fr.z), bf16hi(fr.z), bf16lo(fr.w), bf16hi(fr.w)};
+        float ss = 0.f, y[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss = fmaf(x[e], x[e], ss);
+        for (int o = 1; o < GS; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        const float rr = 1.0f / sqrtf(ss / (float)a.vdim + eps);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) { y[e] = x[e] * rr; if (first) y[e] = (1.0f - lambda) * y[e] + lambda * f[e]; }
+        if (ok) *reinterpret_cast<uint4*>(crow + KW + c) = make_uint4(pack_bf16x2(y[0], y[1]), pack_bf16x2(y[2], y[3]), pack_bf16x2(y[4], y[5]), pack_bf16x2(y[6], y[7]));
+    }
+    for (int c = tid * 8; c < KW; c += 128 * 8) *reinterpret_cast<uint4*>(crow + c) = *reinterpret_cast<const uint4*>(k + t * ldkv + c);
+}
+
 // The visible keys of a query at position p, in the order every kernel walks them: the kept first positions that the window no longer
 // covers, then the window.  n = count; key(i) = i-th visible position.
 struct WinKeys {
@@ -301,9 +350,11 @@ __global__ void __launch_bounds__(128) hy_win_attention_kernel(HyWinAttn a, cons
     float* mm = part + 4 * NM * VD;              // [4][NM]
     float* ll = mm + 4 * NM;                     // [4][NM]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    for (int i = threadIdx.x; i < NM * D; i += blockDim.x) qs[i] = ldf(q + (long long)t * ldq + (long long)h * NM * D + i) * a.scale;
-    __syncthreads();
     const int seq = r.row_seq[t], pos = r.positions[t];
+    const float qscale = a.rel ? a.scale * win_q_temp(a, pos) : a.scale;
+    for (int i = threadIdx.x; i < NM * D; i += blockDim.x) qs[i] = ldf(q + (long long)t * ldq + (long long)h * NM * D + i) * qscale;
+    __syncthreads();
+    const float* rel = a.rel ? a.rel + (long long)h * a.rel_len : nullptr;
     const int32_t* bt = r.block_tables + (long long)seq * r.max_pages_per_seq;
     const WinKeys wk(pos, a.window, a.keep_first);
     const float slope = win_head_slope(a, h);
@@ -327,6 +378,7 @@ __global__ void __launch_bounds__(128) hy_win_attention_kernel(HyWinAttn a, cons
             d = warp_sum(d);
             if (a.softcap > 0.f) d = a.softcap * tanhf(d / a.softcap);
             d -= slope * (float)(pos - j);
+            if (rel) d += rel[min(pos - j, a.rel_len - 1)];
             const float mn = fmaxf(m[mp], d), corr = expf(m[mp] - mn), p = expf(d - mn);
             l[mp] = l[mp] * corr + p; m[mp] = mn;
 #pragma unroll
@@ -408,7 +460,29 @@ __global__ void __launch_bounds__(128) hy_win_attention_kernel(HyWinAttn a, cons
 // output projection's input.
 // ---------------------------------------------------------------------------------------------------------------------------------
 constexpr int WIN_MQ = 64, WIN_KT = 32;
-template <int MAPS, int NVB, bool MOD>      // MOD: soft cap and / or distance slope on the scores
+// score modifiers of the tensor-core forms: 1: soft cap and / or distance slope, 2: a bias per distance and the query temperature
+constexpr int WIN_MOD_NONE = 0, WIN_MOD_CAP_SLOPE = 1, WIN_MOD_REL = 2;
+constexpr float WIN_LOG2E = 1.4426950408889634f;
+// s (16 rows x 32 keys of one warp, raw products) -> base-2 scores with the distance bias, for rows at p_lo / p_hi (heads' tables rel_lo / rel_hi) and
+// keys from k_first on; d_min .. d_max cover every distance of the tile: where they share a row of the bias table, one lookup per row serves the tile
+__device__ __forceinline__ void win_add_rel(const HyWinAttn& a, float (&s)[4][4], int k_first, int lane, int p_lo, int p_hi, float qs_lo, float qs_hi, const float* rel_lo, const float* rel_hi,
+                                            int d_min, int d_max) {
+    const int last = a.rel_len - 1, d0 = min(max(d_min, 0), last);
+    if (a.rel_run[d0] >= d_max) {
+        const float b_lo = rel_lo[d0] * WIN_LOG2E, b_hi = rel_hi[d0] * WIN_LOG2E;
+#pragma unroll
+        for (int nb = 0; nb < 4; ++nb) { s[nb][0] = fmaf(s[nb][0], qs_lo, b_lo); s[nb][1] = fmaf(s[nb][1], qs_lo, b_lo); s[nb][2] = fmaf(s[nb][2], qs_hi, b_hi); s[nb][3] = fmaf(s[nb][3], qs_hi, b_hi); }
+        return;
+    }
+#pragma unroll
+    for (int nb = 0; nb < 4; ++nb)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+            const int key = k_first + nb * 8 + (lane & 3) * 2 + (c & 1), d = min(max((c < 2 ? p_lo : p_hi) - key, 0), last);
+            s[nb][c] = fmaf(s[nb][c], c < 2 ? qs_lo : qs_hi, (c < 2 ? rel_lo : rel_hi)[d] * WIN_LOG2E);
+        }
+}
+template <int MAPS, int NVB, int MOD>
 __global__ void __launch_bounds__(128) hy_win_attention_mma_kernel(HyWinAttn a, const __nv_bfloat16* __restrict__ q, int ldq, const __nv_bfloat16* __restrict__ cache,
                                                                    const float* __restrict__ sink, const __nv_bfloat16* __restrict__ gate, int ldg,
                                                                    __nv_bfloat16* __restrict__ out, int ldo, float eps, HyRows r, const int32_t* __restrict__ tile_seq,
@@ -467,7 +541,14 @@ __global__ void __launch_bounds__(128) hy_win_attention_mma_kernel(HyWinAttn a, 
     // MOD: the scores are scaled, capped, given their distance penalty and brought to base-2 units right after the product
     const float qscale = MOD ? 1.0f : a.scale * 1.4426950408889634f;
     const float inv_cap = a.softcap > 0.f ? a.scale / a.softcap : 0.f;
-    const float slope_lo = MOD ? win_head_slope(a, g * HG + (q0 + 16 * warp + (lane >> 2)) % HG) : 0.f, slope_hi = MOD ? win_head_slope(a, g * HG + (q0 + 16 * warp + (lane >> 2) + 8) % HG) : 0.f;
+    const int h_lo = g * HG + (q0 + 16 * warp + (lane >> 2)) % HG, h_hi = g * HG + (q0 + 16 * warp + (lane >> 2) + 8) % HG;
+    const float slope_lo = MOD == WIN_MOD_CAP_SLOPE ? win_head_slope(a, h_lo) : 0.f, slope_hi = MOD == WIN_MOD_CAP_SLOPE ? win_head_slope(a, h_hi) : 0.f;
+    float qs_lo = 0.f, qs_hi = 0.f; const float *rel_lo = nullptr, *rel_hi = nullptr;
+    if (MOD == WIN_MOD_REL) {
+        const int last_qi = nq - 1, qi_lo = min(16 * warp + (lane >> 2), last_qi), qi_hi = min(16 * warp + (lane >> 2) + 8, last_qi);
+        qs_lo = a.scale * WIN_LOG2E * win_q_temp(a, qpos_of(qi_lo)); qs_hi = a.scale * WIN_LOG2E * win_q_temp(a, qpos_of(qi_hi));
+        rel_lo = a.rel + (long long)h_lo * a.rel_len; rel_hi = a.rel + (long long)h_hi * a.rel_len;
+    }
     const bool active = 16 * warp < nq;
     const int wp_min = active ? qpos_of(16 * warp) : 0, wp_max = active ? qpos_of(min(16 * warp + 15, nq - 1)) : 0;      // positions of the warp's first and last query slot
     load_tile(0, 0);
@@ -498,7 +579,8 @@ __global__ void __launch_bounds__(128) hy_win_attention_mma_kernel(HyWinAttn a, 
                     ldmatrix_x4(ka + 16 * QP * 2 + ks * 32, b0, b1, b2, b3);
                     mma_bf16_16816(s[2], a0, a1, a2, a3, b0, b1); mma_bf16_16816(s[3], a0, a1, a2, a3, b2, b3);
                 }
-                if (MOD) {
+                if (MOD == WIN_MOD_REL) win_add_rel(a, s, k_first, lane, p_lo, p_hi, qs_lo, qs_hi, rel_lo, rel_hi, wp_min - k_last, wp_max - k_first);
+                if (MOD == WIN_MOD_CAP_SLOPE) {
 #pragma unroll
                     for (int nb = 0; nb < 4; ++nb)
 #pragma unroll
@@ -627,7 +709,7 @@ __global__ void __launch_bounds__(128) hy_win_attention_mma_kernel(HyWinAttn a, 
 // query slot join them in warp order and finish the head (sink, a1 - lambda a2, unit RMS, gate).  Which tiles a warp takes depends on the
 // row's position only.
 constexpr int WIN_DEC_WARPS = 8;
-template <int MAPS, int NVB, bool MOD>
+template <int MAPS, int NVB, int MOD>
 __global__ void __launch_bounds__(256) hy_win_decode_mma_kernel(HyWinAttn a, const __nv_bfloat16* __restrict__ q, int ldq, const __nv_bfloat16* __restrict__ cache,
                                                                 const float* __restrict__ sink, const __nv_bfloat16* __restrict__ gate, int ldg,
                                                                 __nv_bfloat16* __restrict__ out, int ldo, float eps, HyRows r, const int32_t* __restrict__ tile_seq,
@@ -671,7 +753,13 @@ __global__ void __launch_bounds__(256) hy_win_decode_mma_kernel(HyWinAttn a, con
     }
     const float qscale = a.scale * 1.4426950408889634f;
     const float inv_cap = a.softcap > 0.f ? a.scale / a.softcap : 0.f;
-    const float slope_lo = MOD ? win_head_slope(a, g * HG + (q0 + (lane >> 2)) % HG) : 0.f, slope_hi = MOD ? win_head_slope(a, g * HG + (q0 + (lane >> 2) + 8) % HG) : 0.f;
+    const int h_lo = g * HG + (q0 + (lane >> 2)) % HG, h_hi = g * HG + (q0 + (lane >> 2) + 8) % HG;
+    const float slope_lo = MOD == WIN_MOD_CAP_SLOPE ? win_head_slope(a, h_lo) : 0.f, slope_hi = MOD == WIN_MOD_CAP_SLOPE ? win_head_slope(a, h_hi) : 0.f;
+    float qs_lo = 0.f, qs_hi = 0.f; const float *rel_lo = nullptr, *rel_hi = nullptr;
+    if (MOD == WIN_MOD_REL) {
+        qs_lo = a.scale * WIN_LOG2E * win_q_temp(a, max(qpos[lane >> 2], 0)); qs_hi = a.scale * WIN_LOG2E * win_q_temp(a, max(qpos[(lane >> 2) + 8], 0));
+        rel_lo = a.rel + (long long)h_lo * a.rel_len; rel_hi = a.rel + (long long)h_hi * a.rel_len;
+    }
     const int p_lo = qpos[lane >> 2], p_hi = qpos[(lane >> 2) + 8];
     const int kc = QD / 8, nc = kc + VD / 8, step_j = 32 / nc, step_c = 32 % nc, j0 = lane / nc, c0 = lane % nc;      // a lane walks its warp's tile chunks in steps of 32
     for (int it = warp; it < n_it; it += WIN_DEC_WARPS) {
@@ -708,6 +796,7 @@ __global__ void __launch_bounds__(256) hy_win_decode_mma_kernel(HyWinAttn a, con
                 ldmatrix_x4(ka + 16 * QP * 2 + ks * 32, b0, b1, b2, b3);
                 mma_bf16_16816(s[2], a0, a1, a2, a3, b0, b1); mma_bf16_16816(s[3], a0, a1, a2, a3, b2, b3);
             }
+            if (MOD == WIN_MOD_REL) win_add_rel(a, s, kt * WIN_KT, lane, p_lo, p_hi, qs_lo, qs_hi, rel_lo, rel_hi, pos_min - (kt * WIN_KT + WIN_KT - 1), pos_max - kt * WIN_KT);
             float mx_lo = -INFINITY, mx_hi = -INFINITY;
 #pragma unroll
             for (int nb = 0; nb < 4; ++nb)
@@ -715,7 +804,8 @@ __global__ void __launch_bounds__(256) hy_win_decode_mma_kernel(HyWinAttn a, con
                 for (int c = 0; c < 4; ++c) {
                     const int key = kt * WIN_KT + nb * 8 + (lane & 3) * 2 + (c & 1), p = c < 2 ? p_lo : p_hi;
                     const bool vis = key <= p && (p - key < a.window || key < a.keep_first);
-                    if (MOD) {
+                    if (MOD == WIN_MOD_REL) s[nb][c] = vis ? s[nb][c] : -INFINITY;
+                    else if (MOD == WIN_MOD_CAP_SLOPE) {
                         const float v = a.softcap > 0.f ? a.softcap * win_tanh(s[nb][c] * inv_cap) : s[nb][c] * a.scale;
                         s[nb][c] = vis ? (v - (c < 2 ? slope_lo : slope_hi) * (float)(p - key)) * 1.4426950408889634f : -INFINITY;
                     } else
@@ -857,6 +947,17 @@ cudaError_t hy_win_prep(bool f32, const HyWinAttn& a, void* q, int ldq, const vo
                : launch_plain(hy_win_prep_kernel<bf>, dim3(r.T), dim3(128), 0, s, a, (bf*)q, ldq, (const bf*)k, (const bf*)v, ldkv, q_norm_w, k_norm_w, eps, (bf*)cache, r);
 }
 
+cudaError_t hy_win_value_prep(bool f32, const HyWinAttn& a, const void* k, const void* v, int ldkv, const HyValueMix& m, float eps, void* cache, const HyRows& r, cudaStream_t s) {
+    if (r.T <= 0) return cudaSuccess;
+    if (a.maps != 1 || a.qk_norm || !k || !v || (a.q_temp_every > 0 && !a.rel)) return cudaErrorInvalidValue;
+    using bf = __nv_bfloat16;
+    const int gs = a.vdim / 8;
+    if (!f32 && a.vdim % 8 == 0 && gs <= 32 && (gs & (gs - 1)) == 0 && (a.kv_heads * a.dim) % 8 == 0 && ldkv % 8 == 0 && (!m.first || (m.first_row % 8 == 0 && m.first_col % 8 == 0)) &&
+        ((reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v) | reinterpret_cast<uintptr_t>(m.first) | reinterpret_cast<uintptr_t>(cache)) & 15) == 0)      // by the model's sizes alone
+        return launch_plain(hy_win_value_prep_vec8_kernel, dim3(r.T), dim3(128), 0, s, a, (const bf*)k, (const bf*)v, ldkv, (const bf*)m.first, m.first_row, m.first_col, m.lambda, eps, (bf*)cache, r);
+    return f32 ? launch_plain(hy_win_value_prep_kernel<float>, dim3(r.T), dim3(128), 0, s, a, (const float*)k, (const float*)v, ldkv, (const float*)m.first, m.first_row, m.first_col, m.lambda, eps, (float*)cache, r)
+               : launch_plain(hy_win_value_prep_kernel<bf>, dim3(r.T), dim3(128), 0, s, a, (const bf*)k, (const bf*)v, ldkv, (const bf*)m.first, m.first_row, m.first_col, m.lambda, eps, (bf*)cache, r);
+}
 cudaError_t hy_win_rope_prep(bool f32, const HyWinAttn& a, const HyRotary& rot, void* q, int ldq, const void* k, const void* v, int ldkv, void* cache, const HyRows& r, cudaStream_t s) {
     if (a.maps != 1 || a.qk_norm || (rot.dims & 1) || rot.dims > a.dim || (rot.v_cos && (a.vdim & 1))) return cudaErrorInvalidValue;
     return f32 ? launch_plain(hy_win_rope_prep_kernel<float>, dim3(r.T), dim3(128), 0, s, a, rot, (float*)q, ldq, (const float*)k, (const float*)v, ldkv, (float*)cache, r)
@@ -909,10 +1010,10 @@ cudaError_t hy_win_attention(bool f32, const HyWinAttn& a, const void* q, int ld
 
 static bool win_modded(const HyWinAttn& a) { return a.softcap > 0.f || a.slope_exp > 0.f; }
 bool hy_win_mma_supported(const HyWinAttn& a) {
-    const bool vd_ok = a.vdim == 16 || a.vdim == 32 || a.vdim == 64 || a.vdim == 96 || a.vdim == 128;
-    return hy_win_supported(a) && a.dim % 16 == 0 && a.dim <= 128 && vd_ok && !(win_modded(a) && a.maps != 1) && a.out_rot != 2;      // score modifiers on the tensor cores: one map; outputs turned back in pairs of neighbours only
+    const bool vd_ok = a.vdim == 16 || a.vdim == 32 || a.vdim == 64 || a.vdim == 96 || a.vdim == 128 || (a.rel && (a.vdim == 48 || a.vdim == 80));
+    return hy_win_supported(a) && a.dim % 16 == 0 && a.dim <= 128 && vd_ok && !((win_modded(a) || a.rel) && a.maps != 1) && !(win_modded(a) && a.rel) && a.out_rot != 2;      // score modifiers on the tensor cores: one map; outputs turned back in pairs of neighbours only
 }
-template <int MAPS, int NVB, bool MOD>
+template <int MAPS, int NVB, int MOD>
 static cudaError_t win_mma_launch(const HyWinAttn& a, const void* q, int ldq, const void* cache, const float* sink, const void* gate, int ldg, void* out, int ldo, float eps,
                                   const HyRows& r, const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles, cudaStream_t s) {
     using bf = __nv_bfloat16;
@@ -927,7 +1028,7 @@ static cudaError_t win_mma_launch(const HyWinAttn& a, const void* q, int ldq, co
     return launch_plain(hy_win_attention_mma_kernel<MAPS, NVB, MOD>, dim3(n_tiles, a.kv_heads), dim3(128), smem, s, a, (const bf*)q, ldq, (const bf*)cache, sink, (const bf*)gate, ldg,
                         (bf*)out, ldo, eps, r, tile_seq, tile_q0);
 }
-template <int MAPS, int NVB, bool MOD>
+template <int MAPS, int NVB, int MOD>
 static cudaError_t win_decode_launch(const HyWinAttn& a, const void* q, int ldq, const void* cache, const float* sink, const void* gate, int ldg, void* out, int ldo, float eps,
                                      const HyRows& r, const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles, cudaStream_t s) {
     using bf = __nv_bfloat16;
@@ -947,26 +1048,32 @@ cudaError_t hy_win_attention_mma(const HyWinAttn& a, const void* q, int ldq, con
                                  const HyRows& r, const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles, cudaStream_t s) {
     if (n_tiles <= 0) return cudaSuccess;
     if (!hy_win_mma_supported(a)) return cudaErrorInvalidValue;
-#define WIN_CASE(M, N) if (a.maps == M && a.vdim == N * 8) return win_mma_launch<M, N, false>(a, q, ldq, cache, sink, gate, ldg, out, ldo, eps, r, tile_seq, tile_q0, n_tiles, s)
-#define WIN_CASE_MOD(N) if (a.vdim == N * 8) return win_mma_launch<1, N, true>(a, q, ldq, cache, sink, gate, ldg, out, ldo, eps, r, tile_seq, tile_q0, n_tiles, s)
+#define WIN_CASE(M, N) if (a.maps == M && a.vdim == N * 8) return win_mma_launch<M, N, WIN_MOD_NONE>(a, q, ldq, cache, sink, gate, ldg, out, ldo, eps, r, tile_seq, tile_q0, n_tiles, s)
+#define WIN_CASE_MOD(N) if (a.vdim == N * 8) return win_mma_launch<1, N, WIN_MOD_CAP_SLOPE>(a, q, ldq, cache, sink, gate, ldg, out, ldo, eps, r, tile_seq, tile_q0, n_tiles, s)
     if (win_modded(a)) { WIN_CASE_MOD(2); WIN_CASE_MOD(4); WIN_CASE_MOD(8); WIN_CASE_MOD(12); WIN_CASE_MOD(16); return cudaErrorInvalidValue; }
+#define WIN_CASE_REL(N) if (a.vdim == N * 8) return win_mma_launch<1, N, WIN_MOD_REL>(a, q, ldq, cache, sink, gate, ldg, out, ldo, eps, r, tile_seq, tile_q0, n_tiles, s)
+    if (a.rel) { WIN_CASE_REL(2); WIN_CASE_REL(4); WIN_CASE_REL(6); WIN_CASE_REL(8); WIN_CASE_REL(10); WIN_CASE_REL(12); WIN_CASE_REL(16); return cudaErrorInvalidValue; }
     WIN_CASE(1, 2); WIN_CASE(1, 4); WIN_CASE(1, 8); WIN_CASE(1, 12); WIN_CASE(1, 16);
     WIN_CASE(2, 2); WIN_CASE(2, 4); WIN_CASE(2, 8); WIN_CASE(2, 12); WIN_CASE(2, 16);
 #undef WIN_CASE
 #undef WIN_CASE_MOD
+#undef WIN_CASE_REL
     return cudaErrorInvalidValue;
 }
 cudaError_t hy_win_decode_mma(const HyWinAttn& a, const void* q, int ldq, const void* cache, const float* sink, const void* gate, int ldg, void* out, int ldo, float eps,
                               const HyRows& r, const int32_t* tile_seq, const int32_t* tile_q0, int n_tiles, cudaStream_t s) {
     if (n_tiles <= 0) return cudaSuccess;
     if (!hy_win_mma_supported(a)) return cudaErrorInvalidValue;
-#define WIN_CASE(M, N) if (a.maps == M && a.vdim == N * 8) return win_decode_launch<M, N, false>(a, q, ldq, cache, sink, gate, ldg, out, ldo, eps, r, tile_seq, tile_q0, n_tiles, s)
-#define WIN_CASE_MOD(N) if (a.vdim == N * 8) return win_decode_launch<1, N, true>(a, q, ldq, cache, sink, gate, ldg, out, ldo, eps, r, tile_seq, tile_q0, n_tiles, s)
+#define WIN_CASE(M, N) if (a.maps == M && a.vdim == N * 8) return win_decode_launch<M, N, WIN_MOD_NONE>(a, q, ldq, cache, sink, gate, ldg, out, ldo, eps, r, tile_seq, tile_q0, n_tiles, s)
+#define WIN_CASE_MOD(N) if (a.vdim == N * 8) return win_decode_launch<1, N, WIN_MOD_CAP_SLOPE>(a, q, ldq, cache, sink, gate, ldg, out, ldo, eps, r, tile_seq, tile_q0, n_tiles, s)
     if (win_modded(a)) { WIN_CASE_MOD(2); WIN_CASE_MOD(4); WIN_CASE_MOD(8); WIN_CASE_MOD(12); WIN_CASE_MOD(16); return cudaErrorInvalidValue; }
+#define WIN_CASE_REL(N) if (a.vdim == N * 8) return win_decode_launch<1, N, WIN_MOD_REL>(a, q, ldq, cache, sink, gate, ldg, out, ldo, eps, r, tile_seq, tile_q0, n_tiles, s)
+    if (a.rel) { WIN_CASE_REL(2); WIN_CASE_REL(4); WIN_CASE_REL(6); WIN_CASE_REL(8); WIN_CASE_REL(10); WIN_CASE_REL(12); WIN_CASE_REL(16); return cudaErrorInvalidValue; }
     WIN_CASE(1, 2); WIN_CASE(1, 4); WIN_CASE(1, 8); WIN_CASE(1, 12); WIN_CASE(1, 16);
     WIN_CASE(2, 2); WIN_CASE(2, 4); WIN_CASE(2, 8); WIN_CASE(2, 12); WIN_CASE(2, 16);
 #undef WIN_CASE
 #undef WIN_CASE_MOD
+#undef WIN_CASE_REL
     return cudaErrorInvalidValue;
 }
 

@@ -18,7 +18,7 @@ int make_tmap_bf16_2d(CUtensorMap* out, const void* base, uint64_t rows, uint64_
 enum GemmEpilogue : int {
     EPI_STORE = 0,    // out[M,N] bf16 = act(acc (+ bias[N])), act = identity, relu(.)^2 or the tanh form of GELU (GemmParams::store_act)
     EPI_RESID = 1,    // out[M,N] bf16 = acc + resid[M,N]      (out may alias resid)
-    EPI_SWIGLU = 2,   // out[M,N/2] bf16 = silu(gate)*up, B rows interleaved 16 gate / 16 up
+    EPI_SWIGLU = 2,   // out[M,N/2] bf16 = silu(gate)*up, B rows interleaved 16 gate / 16 up; GemmParams::glu_limit > 0: the clamped gated activation, rows scaled before it
     EPI_LOGITS = 3,   // per-row (max, argmax) partial per N-tile -> argmax_ws; optional fp32 logits store
     EPI_F32 = 4,      // f32_out[M,N] fp32 = alpha * acc (+ bias_f32[N]) (+ f32_out when f32_accumulate): fp32 residual streams and logits
 };
@@ -37,6 +37,9 @@ struct GemmParams {
     // grouped product (routed experts): row tile m uses the B rows of group m_tile_group[m] (B = the groups' [group_rows, K] matrices stacked);
     // row tiles >= *n_m_tiles do nothing.  Both live on the device and may come from the preceding kernel.
     const int32_t* m_tile_group; const int32_t* n_m_tiles; int group_rows;
+    // EPI_SWIGLU with glu_limit > 0: out = g sigmoid(glu_slope g) (u + 1), g = min(s gate, limit), u = clamp(s up, -limit, limit), where row r's s is
+    // row_scale[row_scale_idx[r]] (0 for a negative index: a padding row of a grouped product) — the router's weight on an expert's input, exact in fp32
+    float glu_limit, glu_slope; const float* row_scale; const int32_t* row_scale_idx;
 };
 // tmA: box {64, 128} over A[M,K]; tmB: box {64, block_n} over B[N,K].  block_n in {32,64,128,256}.
 cudaError_t launch_gemm(const CUtensorMap* tmA, const CUtensorMap* tmB, const GemmParams& p, int epilogue, int block_n,

@@ -1,8 +1,9 @@
-"""Throughput of the hybrid family beside the closest existing models (`bench.py --arch ratasun | zurevik | rofizen | gosavik`): Ratasun beside the
+"""Throughput of the hybrid family beside the closest existing models (`bench.py --arch ratasun | zurevik | rofizen | gosavik | petipel`): Ratasun beside the
 Llama-family model of equal width, depth and active feed-forward size; Zurevik and Rofizen beside the Ratasun model of equal width, depth and
 experts (the closest design: routed experts in every layer; recurrent mixers with an fp32 state like Rofizen's) and beside that Llama-family model;
 Gosavik (dense feed-forward, attention mixers only) beside the Llama-family model of equal width, depth and feed-forward size — the closest model as a whole —
-and beside Ratasun, whose latent attention is the closest kernel to its own.  Random weights (seeded on load), synthetic token ids; prefill = real chunked prefill of batch x (ctx-1) tokens,
+and beside Ratasun, whose latent attention is the closest kernel to its own; Petipel (linear attention with a gate per key channel, cached-key/value
+attention, routed experts) beside Rofizen, which has the closest kernel for each of its own, and beside both of those.  Random weights (seeded on load), synthetic token ids; prefill = real chunked prefill of batch x (ctx-1) tokens,
 decode = steps of the whole batch, both timed with CUDA events inside the engine (oa_bench_decode).  With --breakdown the per-kernel-class
 device times come from the engine's in-situ event timing (OA_PROFILE_ALL), one pass for prefill and one for decode."""
 from __future__ import annotations
@@ -88,6 +89,23 @@ def gosavik_sizes(name: str) -> dict:
             "layers": [{"type": t, "mixer": m, "mlp": mlp} for t, m in order]}
 
 
+def petipel_sizes(name: str) -> dict:
+    """Petipel at the width, depth (6 layers) and feed-forward sizes of rofizen_sizes(name): three HGRN2 layers with a dense feed-forward alternate with
+    three attention layers that route each token to 4 experts."""
+    if name == "small":
+        heads, dim, vdim, width, ff, experts = 8, 64, 128, 1024, 512, 16
+        att = {"heads": 16, "kv_heads": 4, "dim": 64, "vdim": 64, "scale": 64 ** -0.5}
+    else:
+        heads, dim, vdim, width, ff, experts = 16, 128, 128, 2048, 1024, 32
+        att = {"heads": 16, "kv_heads": 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
+    att.update(bias_max=128, v_mix=True, q_temp={"coef": 0.1, "every": 256})
+    rec = {"heads": heads, "dim": dim, "vdim": vdim}
+    dense = {"kind": "dense", "ff": 4 * ff}
+    moe = {"kind": "moe", "expert": {"ff": ff, "limit": 7.0}, "router": {"experts": experts, "top": 4}}
+    return {"architecture": "Petipel", "width": width, "vocab": 32000, "norm": {"eps": 1e-5}, "residual_mult": 0.5,
+            "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in [("hgrn2", rec, dense), ("attention", att, moe)] * 3]}
+
+
 def one(engine_cfg: dict, batch: int, ctx: int, steps: int, warmup: int, breakdown: bool) -> dict:
     from .engine import Engine
     out = {}
@@ -113,7 +131,7 @@ def one(engine_cfg: dict, batch: int, ctx: int, steps: int, warmup: int, breakdo
 
 
 def run(args) -> None:
-    zu = args.arch in ("zurevik", "rofizen", "gosavik")
+    zu = args.arch in ("zurevik", "rofizen", "gosavik", "petipel")
     res = {"metric": args.arch + "_vs_ratasun_and_llama_throughput" if zu else "hybrid_vs_llama_throughput", "unit": "tokens/s", "data": "synthetic", "dtype": "bf16", "cases": []}
     for name in args.arch_sizes.split(","):
         sz = sizes(name)
@@ -128,12 +146,16 @@ def run(args) -> None:
                 return one(dict(common, model_dir=d, **json.loads(args.engine_extra)), batch, ctx, args.steps, args.warmup, args.breakdown)
         case = {"size": name, "batch": batch, "ctx": ctx, "layer_runs": sz["runs"]}
         if zu:
-            case[args.arch] = folder_model({"zurevik": zurevik_sizes, "rofizen": rofizen_sizes, "gosavik": gosavik_sizes}[args.arch](name))
+            case[args.arch] = folder_model({"zurevik": zurevik_sizes, "rofizen": rofizen_sizes, "gosavik": gosavik_sizes, "petipel": petipel_sizes}[args.arch](name))
+        if args.arch == "petipel":
+            case["rofizen"] = folder_model(rofizen_sizes(name))
         case["ratasun"] = hy = folder_model(sz["hybrid"])
         case["llama_equal_size"] = ll = one(dict(common, **sz["llama"]), batch, ctx, args.steps, args.warmup, args.breakdown)
         new = case[args.arch] if zu else hy
         case["prefill_ratio"], case["decode_ratio"] = new["prefill_tok_s"] / ll["prefill_tok_s"], new["decode_tok_s"] / ll["decode_tok_s"]
         if zu:
+            if args.arch == "petipel":
+                case["prefill_ratio_to_rofizen"], case["decode_ratio_to_rofizen"] = (new[k] / case["rofizen"][k] for k in ("prefill_tok_s", "decode_tok_s"))
             case["prefill_ratio_to_ratasun"], case["decode_ratio_to_ratasun"] = new["prefill_tok_s"] / hy["prefill_tok_s"], new["decode_tok_s"] / hy["decode_tok_s"]
         res["cases"].append(case)
     print(json.dumps(res))

@@ -32,7 +32,7 @@ OA_DEVINL float gelu_tanh_f32(float z) { return 0.5f * z * (1.0f + tanhf(0.79788
 // gated activation with clamped halves: g sigmoid(slope g) (u + 1), g = min(g, limit), u in [-limit, limit]
 OA_DEVINL float clamped_glu_f32(float g, float u, float limit, float slope) {
     g = fminf(g, limit); u = fminf(fmaxf(u, -limit), limit);
-    return g / (1.0f + __expf(-slope * g)) * (u + 1.0f);
+    return __fdividef(g, 1.0f + __expf(-slope * g)) * (u + 1.0f);
 }
 OA_DEVINL uint32_t pack_bf16x2(float a, float b) {
     uint32_t r;

@@ -444,9 +444,12 @@ __global__ void __launch_bounds__(GEMM_THREADS, 1) gemm_persistent_kernel(const 
         for (int t = blockIdx.x; t < total_tiles; t += gridDim.x, ++it) {
             int m_blk, n_blk; raster_tile(t, m_tiles, n_tiles, m_blk, n_blk);
             const int as = it & 1;
+            const int row_base = m_blk * BLOCK_M + q * 32;
+            float glu_sc[2] = {0.f, 0.f};          // scales of the two rows this lane stores (clamped gated activation), read while the tile is still being multiplied
+            if (EPI == EPI_SWIGLU && p.glu_limit > 0.f)
+                for (int i2 = 0; i2 < 2; ++i2) if (row_base + i2 * 16 + (lane >> 1) < p.M) glu_sc[i2] = glu_row_scale(p, row_base + i2 * 16 + (lane >> 1));
             mbar_wait(&acc_full[as], ((uint32_t)it >> 1) & 1);
             tcgen05_fence_after();
-            const int row_base = m_blk * BLOCK_M + q * 32;
 #pragma unroll 1
             for (int cc = 0; cc < BN; cc += 32) {
                 uint32_t v[32];
@@ -471,9 +474,8 @@ __global__ void __launch_bounds__(GEMM_THREADS, 1) gemm_persistent_kernel(const 
                         const float uu[8] = {u0.x, u0.y, u0.z, u0.w, u1.x, u1.y, u1.z, u1.w};
                         float f[8];
                         if (p.glu_limit > 0.f) {
-                            const float sc = row < p.M ? glu_row_scale(p, row) : 0.f;
 #pragma unroll
-                            for (int k = 0; k < 8; ++k) f[k] = clamped_glu_f32(gg[k] * sc, uu[k] * sc, p.glu_limit, p.glu_slope);
+                            for (int k = 0; k < 8; ++k) f[k] = clamped_glu_f32(gg[k] * glu_sc[i2], uu[k] * glu_sc[i2], p.glu_limit, p.glu_slope);
                         } else
 #pragma unroll
                         for (int k = 0; k < 8; ++k) f[k] = __fdividef(gg[k], 1.0f + __expf(-gg[k])) * uu[k];

@@ -187,6 +187,13 @@ cudaError_t hy_lin_prep(bool f32, const HyLinPrep& p, const void* q, const void*
 // (its own evaluation: no cancellation where the gate is nearly open), v -> vv; lower, bias [heads * dim] fp32
 cudaError_t hy_forget_prep(bool f32, int heads, int dim, int vdim, const void* q, const void* z, const void* v, int ld, const float* bias, const float* lower, float* qq, float* kk, float* vv,
                            float* dec, int T, cudaStream_t s);
+// The same, the recurrence S <- diag(f) S + (1 - f) v^T, o = S^T q and the per-head RMS norm (weight [vdim] shared by heads) in one kernel (bf16; sizes
+// below): out [T, ldo] = the heads' normed read-outs, the output projection's input.  state as hy_recurrence keeps it.  few / many: whether the step has
+// sequences of at most / of more than HY_FORGET_FEW_ROWS rows (token by token / blocks of tokens on the tensor cores)
+constexpr int HY_FORGET_FEW_ROWS = 4;
+bool hy_forget_mix_supported(int dim, int vdim);        // multiples of 8 up to 128
+cudaError_t hy_forget_mix(int heads, int dim, int vdim, const void* q, const void* z, const void* v, int ld, const float* bias, const float* lower, const float* norm_w, float eps, float* state,
+                          void* out, int ldo, bool few, bool many, const HyRows& r, cudaStream_t s);
 // Matrix memory.  gates [T, ldg] fp32 = [W_i h + b_i | W_f h + b_f] (heads each).  hy_mlstm_gates: log gates i = cap tanh(. / cap),
 // f = logsigmoid(cap tanh(. / cap)); the running maximum m_t = max(f_t + m_(t-1), i_t) per (sequence, head), carried in mstate [slots, heads]
 // (a sequence whose step starts at position 0 starts from m = 0); out: dec[t, h] = exp(f + m_(t-1) - m_t), gin[t, h] = exp(i - m_t), floor_[t, h] = exp(-m_t)

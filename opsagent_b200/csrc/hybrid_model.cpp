@@ -641,6 +641,10 @@ void HybridModel::linear_mixer(const HyRun& run, const HyLayer& l, const LayerW&
         cuda_check(hy_recurrence(HY_REC_CHANNEL, qq_, kk_, vv_, dec_, nullptr, rec_, st, H, H, D, VD, r, stream), "gated linear attention"); MARK(8);
         cuda_check(hy_gated_norm(f32_, rec_, H * VD, VD, w.norm_w, VD, g, ld_proj_, 0, n.gate_silu, nullptr, 1, nullptr, 0, mix_, ld_mix_, hc_.eps, T, stream), "gated norm"); MARK(9);
     } else if (n.kind == HY_LIN_FORGET_WRITE) {
+        if (!f32_ && opt.hy_tensor_core && hy_forget_mix_supported(D, VD)) {       // by the model's sizes alone; hy_tensor_core = 0 takes the separate kernels
+            cuda_check(hy_forget_mix(H, D, VD, q, k, v, ld_proj_, w.f_bias, w.f_lower, w.norm_w, hc_.eps, st, mix_, ld_mix_, few_rows_, many_rows_, r, stream), "forget-gate mixer"); MARK(8);
+            return;
+        }
         cuda_check(hy_forget_prep(f32_, H, D, VD, q, k, v, ld_proj_, w.f_bias, w.f_lower, qq_, kk_, vv_, dec_, T, stream), "forget gate operands"); MARK(28);
         cuda_check(hy_recurrence(HY_REC_CHANNEL, qq_, kk_, vv_, dec_, nullptr, rec_, st, H, H, D, VD, r, stream), "forget-gate recurrence"); MARK(8);
         cuda_check(hy_gated_norm(f32_, rec_, H * VD, VD, w.norm_w, VD, nullptr, 4, 0, 0, nullptr, 1, nullptr, 0, mix_, ld_mix_, hc_.eps, T, stream), "head norm"); MARK(9);
@@ -809,11 +813,12 @@ void HybridModel::forward(const StepInput& in, float* logits_out) {
     const int T = (int)in.tokens.size(), S = in.n_seqs, NS = (int)in.sample_rows.size(), W = hc_.width, V = hc_.vocab;
     if (T <= 0 || T > MR_ || NS > MS_ || S <= 0 || S > opt.max_batch) throw std::runtime_error("forward: bad batch size");
     if ((int)in.seq_row0.size() != S + 1 || (int)in.state_slots.size() != S || in.seq_row0[S] != T) throw std::runtime_error("forward: this model needs the rows of every sequence (seq_row0) and its state slot");
-    row_seq_.resize(T); seq_pos0_.resize(S);
+    row_seq_.resize(T); seq_pos0_.resize(S); few_rows_ = many_rows_ = false;
     for (int s = 0; s < S; ++s) {
         if (in.seq_row0[s + 1] <= in.seq_row0[s]) throw std::runtime_error("forward: empty sequence in a step");
         if (state_slots > 0 && (in.state_slots[s] < 0 || in.state_slots[s] >= state_slots)) throw std::runtime_error("forward: state slot out of range");
         seq_pos0_[s] = in.positions[in.seq_row0[s]];
+        (in.seq_row0[s + 1] - in.seq_row0[s] <= HY_FORGET_FEW_ROWS ? few_rows_ : many_rows_) = true;
         for (int t = in.seq_row0[s]; t < in.seq_row0[s + 1]; ++t) { row_seq_[t] = s; if (in.positions[t] != seq_pos0_[s] + (t - in.seq_row0[s])) throw std::runtime_error("forward: rows of a sequence must be consecutive positions"); }
         if (in.positions[in.seq_row0[s + 1] - 1] >= opt.max_seq_len) throw std::runtime_error("forward: position beyond max_seq_len");
     }

@@ -105,6 +105,7 @@ private:
     float *xs_ = nullptr, *hn_ = nullptr, *shift_prev_ = nullptr, *ones_ = nullptr; void* cq_ = nullptr; int ld_cq_ = 0, n_streams_ = 1;      // residual streams [T, n, W]; normed rows before the shift; carried rows of the step's sequences
     std::vector<float*> aux_;                      // per matrix-memory execution: [slots][heads * dim] normaliser, then [slots][heads] running maximum
     int MR_ = 0, MS_ = 0, Wld_ = 0;
+    bool few_rows_ = false, many_rows_ = false;    // the step has sequences of at most / of more than HY_FORGET_FEW_ROWS rows
     // activations
     float *x_ = nullptr, *x0_ = nullptr, *q_abs_ = nullptr, *qq_ = nullptr, *kk_ = nullptr, *vv_ = nullptr, *dec_ = nullptr, *beta_ = nullptr, *rec_ = nullptr, *wgt_ = nullptr,
           *logits_ = nullptr, *moe_y_ = nullptr, *rlog_ = nullptr;

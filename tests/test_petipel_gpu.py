@@ -337,9 +337,9 @@ TC_STACKS = {
     "buckets_inside_tiles": [A(heads=4, kv_heads=2, dim=32, vdim=48, reach=100, rows=32, mlp=D(96)), H(heads=2, dim=32, vdim=64, mlp=M(experts=8, top=2, ff=32)),
                              A(heads=8, kv_heads=2, dim=16, vdim=48, reach=400, rows=12, q_temp=(0.3, 100))],
     "large_group_and_wide_heads": [A(heads=20, kv_heads=1, dim=64, vdim=128, reach=600, rows=24, scale=0.1, q_temp=None), A(heads=6, kv_heads=1, dim=16, vdim=128, reach=30, rows=32, mlp=M(experts=5, top=1, ff=48)),
-                                   H(heads=1, dim=128, vdim=96)],
+                                   H(heads=1, dim=128, vdim=96), H(heads=2, dim=96, vdim=24)],
     "one_head_per_group_and_other_widths": [A(heads=3, kv_heads=3, dim=48, vdim=80, reach=50, rows=7, mlp=D(64)), A(heads=2, kv_heads=2, dim=128, vdim=96, reach=64, rows=16, v_mix=False),
-                                            A(heads=2, kv_heads=1, dim=16, vdim=32, v_mix=False), A(heads=2, kv_heads=1, dim=16, vdim=64, v_mix=False, reach=33)],
+                                            H(heads=2, dim=40, vdim=88), H(heads=1, dim=16, vdim=128), A(heads=2, kv_heads=1, dim=16, vdim=32, v_mix=False), A(heads=2, kv_heads=1, dim=16, vdim=64, v_mix=False, reach=33)],
 }
 
 

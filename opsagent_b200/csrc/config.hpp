@@ -69,7 +69,7 @@ struct ModelConfig {
     float init_std = 0.02f;
     uint64_t seed = 1234;
     std::string chat_template = "llama3";   // or "chatml"
-    // model registry key: "llama" (Llama-3 / Qwen2.5 decoders, the fields above) or a design of the hybrid family, "ratasun" / "zurevik" (sizes in
+    // model registry key: "llama" (Llama-3 / Qwen2.5 decoders, the fields above) or a design of the hybrid family, "ratasun" / "zurevik" / "rofizen" / "gosavik" / "petipel" (sizes in
     // `hybrid`, read from the checkpoint folder's config.json, whose "architecture" key selects the class)
     std::string arch = "llama";
     std::shared_ptr<HybridConfig> hybrid;

@@ -12,7 +12,7 @@
 // latent attention with a low-rank query, rotate-half rotary with YaRN-scaled frequencies, a sliding window, a sink and a per-channel output
 // gate, or causal grouped-query attention with projection biases, short convolutions on q / k / v, interleaved rotary, rotated values
 // and a sink; feed-forward: dense with the tanh form of GELU.  "Petipel": sublayers in sequence with an RMS norm on either side of each
-// (x += m norm(sublayer(norm(x))), weights stored around zero); mixers: causal grouped-query attention without rotation (a learned bias per
+// (x += m norm(sublayer(norm(x))), factors stored as w - 1); mixers: causal grouped-query attention without rotation (a learned bias per
 // head and distance bucket on the scores, a query temperature, values of unit RMS that later layers mix with the first layer's, a gate per
 // head), or HGRN2 (a recurrence that writes with the complement of its forget gate); feed-forward: dense with PolyNorm, or experts with a
 // clamped gated activation that are chosen by, and read their input times, a sigmoid score.
@@ -64,7 +64,7 @@ struct HyMoe {
     int router = HY_ROUTER_SIGMOID_GROUPS, act = HY_EXPERT_SWIGLU;
     bool dense = false;                   // one feed-forward for every token (no router, no experts): down(act(up h)), width ff
     float limit = 0.f;                    // clamped gated activation
-    bool weight_on_input = false;         // the router's weight multiplies the expert's input, not its output
+    bool weight_on_input = false;         // an expert reads weight * h, and its output is added as it is
     int shared_ff = 0;                    // > 0: a shared expert of this width runs for every token, times sigmoid(w_sg . h)
 };
 

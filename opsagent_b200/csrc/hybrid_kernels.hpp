@@ -7,6 +7,9 @@
 // token ids) and the routed experts (SwiGLU; squared ReLU); several residual streams joined by learned coefficients with the RMS norm that
 // opens a sublayer, the token shift, rotary preparation of cached keys and values (also fused with short convolutions), rotated values and
 // the counter-rotation of the heads' outputs, window / sink / gate on latent attention (hybrid_streams.cu, hybrid_window.cu, hybrid_kernels.cu).
+// Norms on both sides of a sublayer, PolyNorm (hybrid_streams.cu); a learned bias per distance on the scores, unit-RMS values mixed with another
+// layer's (hybrid_window.cu); the recurrence that writes with the complement of its forget gate, alone and fused with its gates and its norm
+// (hybrid_linear.cu); a router of plain sigmoids and experts with a clamped gated activation and a weight on their input (hybrid_kernels.cu).
 // Each mechanism takes its sizes and constants as arguments.
 //
 // `f32` selects the activation / matrix element type: false = bf16 storage with fp32 accumulation, true = everything in fp32.  What must be

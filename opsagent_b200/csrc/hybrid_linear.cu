@@ -454,8 +454,8 @@ template <int CV> __device__ __forceinline__ void load_cv(const __nv_bfloat16* p
 #pragma unroll
     for (int e = 0; e < CV; e += 4) { const uint2 x = *reinterpret_cast<const uint2*>(p + e); f[e] = bf16lo(x.x); f[e + 1] = bf16hi(x.x); f[e + 2] = bf16lo(x.y); f[e + 3] = bf16hi(x.y); }
 }
-template <int DP, int THREADS>
-__global__ void __launch_bounds__(THREADS, 2) hy_forget_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ z, const __nv_bfloat16* __restrict__ v, int ld,
+template <int DP, int THREADS, int CTAS>      // CTAS per SM the registers are cut for: 2, or 1 where the grid does not fill the SMs once (the same arithmetic)
+__global__ void __launch_bounds__(THREADS, CTAS) hy_forget_chunk_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ z, const __nv_bfloat16* __restrict__ v, int ld,
                                                                      const float* __restrict__ bias, const float* __restrict__ lower, const float* __restrict__ norm_w, float* __restrict__ state,
                                                                      __nv_bfloat16* __restrict__ out, int ldo, int H, int D, int VD, float eps, HyRows r) {
     HY_PDL();
@@ -730,7 +730,7 @@ cudaError_t hy_forget_mix(int heads, int dim, int vdim, const void* q, const voi
     const size_t raw = (size_t)2 * FW_TB * (2 * dim + vdim + 8) * 2, smem_few = (size_t)FW_TB * (3 * dp + vp) * 4 + raw;
     const size_t smem_many = ((size_t)FW_TB * (3 * dp + vp + 4) + 3 * dp + vp) * 4 + (size_t)FW_TB * (3 * (dp + 8) + 2 * (FW_TB + 8)) * 2 + raw;
     const dim3 grid(r.S, heads);
-    static bool done[6][16] = {};
+    static bool done[7][16] = {};
     auto go = [&](auto kern, bool (&flag)[16], int threads, size_t smem) -> cudaError_t {
         if (cudaError_t e = ensure_dynamic_smem(kern, 100 * 1024, flag); e != cudaSuccess) return e;
         return launch_plain(kern, grid, dim3(threads), smem, s, (const bf*)q, (const bf*)z, (const bf*)v, ld, bias, lower, norm_w, state, (bf*)out, ldo, heads, dim, vdim, eps, r);
@@ -739,9 +739,12 @@ cudaError_t hy_forget_mix(int heads, int dim, int vdim, const void* q, const voi
         const cudaError_t e = dp == 64 ? go(hy_forget_mix_kernel<1>, done[0], std::max(64, vp * 2), smem_few) : go(hy_forget_mix_kernel<2>, done[1], std::max(64, vp * 2), smem_few);
         if (e != cudaSuccess) return e;
     }
-    if (many) {          // a token's 8-channel pieces are a power of two of threads
-        const cudaError_t e = vp <= 64 ? (dp == 64 ? go(hy_forget_chunk_kernel<64, 128>, done[2], 128, smem_many) : go(hy_forget_chunk_kernel<128, 128>, done[3], 128, smem_many))
-                                       : (dp == 64 ? go(hy_forget_chunk_kernel<64, 256>, done[4], 256, smem_many) : go(hy_forget_chunk_kernel<128, 256>, done[5], 256, smem_many));
+    if (many) {
+        static int sms = 0;
+        if (!sms) { int dev = 0; cudaGetDevice(&dev); if (cudaError_t e = cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev); e != cudaSuccess) return e; }
+        // a token's 8-channel pieces are a power of two of threads
+        const cudaError_t e = vp <= 64 ? (dp == 64 ? go(hy_forget_chunk_kernel<64, 128, 2>, done[2], 128, smem_many) : go(hy_forget_chunk_kernel<128, 128, 2>, done[3], 128, smem_many))
+                                       : (dp == 64 ? go(hy_forget_chunk_kernel<64, 256, 2>, done[4], 256, smem_many) : r.S * heads <= sms ? go(hy_forget_chunk_kernel<128, 256, 1>, done[6], 256, smem_many) : go(hy_forget_chunk_kernel<128, 256, 2>, done[5], 256, smem_many));
         if (e != cudaSuccess) return e;
     }
     return cudaSuccess;

@@ -39,6 +39,8 @@ def steady_routing(cfg, W):
     for name in W:
         if name.endswith(("mix.o", "down")):
             W[name][:8] = 0.0
+        if name.endswith("norm2"):
+            W[name][:8] = 0.0
         if name.endswith("router"):
             assert W[name].shape[0] <= 8
             W[name] = np.roll(np.eye(W[name].shape[0], W[name].shape[1]), int(name[1]), 0)

@@ -26,14 +26,17 @@ __host__ OA_DEVINL uint16_t f32_to_bf16_bits(float f) {
 OA_DEVINL float bf16_bits_to_f32(uint16_t h) { return __uint_as_float(((uint32_t)h) << 16); }
 OA_DEVINL float bf16lo(uint32_t packed) { return __uint_as_float(packed << 16); }
 OA_DEVINL float bf16hi(uint32_t packed) { return __uint_as_float(packed & 0xffff0000u); }
-// pack two fp32 -> bf16x2 (lo = a, hi = b), RNE (cvt.rn.bf16x2.f32 takes hi operand first)
 // the tanh form of GELU: 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))
 OA_DEVINL float gelu_tanh_f32(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+// the same as z sigmoid(2 sqrt(2 / pi) (z + 0.044715 z^3)), from the fast exponential and divide: for values that are rounded to bf16 next
+OA_DEVINL float gelu_tanh_fast_f32(float z) { return __fdividef(z, 1.0f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z))); }
+OA_DEVINL float silu_fast_f32(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
 // gated activation with clamped halves: g sigmoid(slope g) (u + 1), g = min(g, limit), u in [-limit, limit]
 OA_DEVINL float clamped_glu_f32(float g, float u, float limit, float slope) {
     g = fminf(g, limit); u = fminf(fmaxf(u, -limit), limit);
     return __fdividef(g, 1.0f + __expf(-slope * g)) * (u + 1.0f);
 }
+// pack two fp32 -> bf16x2 (lo = a, hi = b), RNE (cvt.rn.bf16x2.f32 takes hi operand first)
 OA_DEVINL uint32_t pack_bf16x2(float a, float b) {
     uint32_t r;
     asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(r) : "f"(b), "f"(a));

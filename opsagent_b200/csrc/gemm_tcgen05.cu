@@ -12,7 +12,7 @@
 //
 // The role of this file in the reference's terms: it is the arithmetic that sits behind
 // llms.OpenAIClient.Chat (reference pkg/llms/openai.go:69-104) once the `local-cuda` provider replaces the
-// remote HTTP server — see DESIGN.md §Kernels.
+// remote HTTP server.
 #include <algorithm>
 #include <cstdlib>
 
@@ -174,6 +174,9 @@ __global__ void __launch_bounds__(GEMM_THREADS) gemm_tcgen05_kernel(const __grid
                             } else if (p.store_act == 2) {
 #pragma unroll
                                 for (int i = 0; i < 8; ++i) f[i] = gelu_tanh_f32(f[i]);
+                            } else if (p.store_act == 3 && col0 + j >= p.act_col0 && col0 + j < p.act_col1) {
+#pragma unroll
+                                for (int i = 0; i < 8; ++i) f[i] = silu_fast_f32(f[i]);
                             }
                             uint4 o;
                             o.x = pack_bf16x2(f[0], f[1]); o.y = pack_bf16x2(f[2], f[3]);
@@ -208,6 +211,9 @@ __global__ void __launch_bounds__(GEMM_THREADS) gemm_tcgen05_kernel(const __grid
                         const float sc = glu_row_scale(p, row);
 #pragma unroll
                         for (int i = 0; i < 16; ++i) f[i] = clamped_glu_f32(__uint_as_float(v[i]) * sc, __uint_as_float(v[16 + i]) * sc, p.glu_limit, p.glu_slope);
+                    } else if (p.glu_gelu) {
+#pragma unroll
+                        for (int i = 0; i < 16; ++i) f[i] = gelu_tanh_fast_f32(__uint_as_float(v[i])) * __uint_as_float(v[16 + i]);
                     } else
 #pragma unroll
                     for (int i = 0; i < 16; ++i) {
@@ -476,6 +482,9 @@ __global__ void __launch_bounds__(GEMM_THREADS, 1) gemm_persistent_kernel(const 
                         if (p.glu_limit > 0.f) {
 #pragma unroll
                             for (int k = 0; k < 8; ++k) f[k] = clamped_glu_f32(gg[k] * glu_sc[i2], uu[k] * glu_sc[i2], p.glu_limit, p.glu_slope);
+                        } else if (p.glu_gelu) {
+#pragma unroll
+                            for (int k = 0; k < 8; ++k) f[k] = gelu_tanh_fast_f32(gg[k]) * uu[k];
                         } else
 #pragma unroll
                         for (int k = 0; k < 8; ++k) f[k] = __fdividef(gg[k], 1.0f + __expf(-gg[k])) * uu[k];
@@ -521,6 +530,9 @@ __global__ void __launch_bounds__(GEMM_THREADS, 1) gemm_persistent_kernel(const 
                                 } else if (p.store_act == 2) {
 #pragma unroll
                                     for (int k = 0; k < 8; ++k) f[k] = gelu_tanh_f32(f[k]);
+                                } else if (p.store_act == 3 && col >= p.act_col0 && col < p.act_col1) {
+#pragma unroll
+                                    for (int k = 0; k < 8; ++k) f[k] = silu_fast_f32(f[k]);
                                 }
                             } else {
                                 const uint4 rr = *reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(p.resid) + (size_t)row * p.ldr + col);

@@ -2,7 +2,7 @@
 // attention (a compressed key/value cache), a gated delta rule with per-channel decay, a Mamba-2 state-space layer, or windowed attention
 // over cached keys and values (sliding window with optional kept first tokens, one or two score maps per head, optional sink, output gate,
 // optionally reading another layer's cache), each beside a routed mixture-of-experts feed-forward, with an optional looped block that
-// re-injects the embedding.  Five designs are registered: "Ratasun" (one weight-only layer norm per layer, sigmoid group-limited router, SwiGLU
+// re-injects the embedding.  Six designs are registered: "Ratasun" (one weight-only layer norm per layer, sigmoid group-limited router, SwiGLU
 // experts), "Zurevik" (two RMS norms per layer, softmax over the chosen router logits, squared-ReLU experts, scaled embedding, soft-capped
 // logits) and "Rofizen" (norm after the sum: x <- norm(alpha x + sublayer(x)), mixer and feed-forward in sequence; mixers: gated linear
 // attention with a decay per key channel, retention with a fixed decay per head and rotate-half rotary, or causal soft-capped attention with
@@ -15,7 +15,11 @@
 // (x += m norm(sublayer(norm(x))), factors stored as w - 1); mixers: causal grouped-query attention without rotation (a learned bias per
 // head and distance bucket on the scores, a query temperature, values of unit RMS that later layers mix with the first layer's, a gate per
 // head), or HGRN2 (a recurrence that writes with the complement of its forget gate); feed-forward: dense with PolyNorm, or experts with a
-// clamped gated activation that are chosen by, and read their input times, a sigmoid score.
+// clamped gated activation that are chosen by, and read their input times, a sigmoid score.  "Ketopel": plain pre-norm sublayers in sequence; mixers:
+// latent attention with a sigmoid gate per head, a gated delta rule with one decay per head, or capped grouped-query attention (one norm over
+// the whole query / key projection, rotate-half rotary with YaRN-scaled frequencies) beside lightning attention (a linear recurrence of activated
+// queries, keys and values with a fixed decay per head, one norm over all heads), joined by two fixed factors; feed-forward: dense, gelu(gate) * up;
+// a looped block that adds the embedding and a learned vector before its passes.
 // Every size and constant is read from the checkpoint folder's config.json; nothing here is specific to one checkpoint.
 #pragma once
 #include <cstdio>
@@ -34,11 +38,11 @@ enum HyNorm : int { HY_LAYER_NORM = 0, HY_RMS_NORM = 1 };
 enum HyRouterKind : int { HY_ROUTER_SIGMOID_GROUPS = 0, HY_ROUTER_SOFTMAX_CHOSEN = 1, HY_ROUTER_TOKEN_TABLE = 2, HY_ROUTER_SIGMOID_CHOSEN = 3 };   // weights: sigmoid scores renormalised and scaled / softmax over the chosen logits / a table row per token id, 1 / top each / the chosen logits' sigmoids as they are
 // linear-attention recurrences over an fp32 state S[dim, vdim] per head, o_t = S_t^T q_t:
 //   channel decay: S_t = diag(a_t) S_(t-1) + k_t v_t^T, a_t = sigmoid(z_t)^(1 / tau) per key channel from a low-rank projection (gated linear attention)
-//   head decay:    S_t = decay_h S_(t-1) + k_t v_t^T with a fixed decay per head, rotate-half rotary on q and k (retention)
+//   head decay:    S_t = decay_h S_(t-1) + k_t v_t^T with a fixed decay per head, rotate-half rotary on q and k (retention), or q = silu(.), k = silu(.), v = silu(.) (lightning attention)
 //   forget write:  S_t = diag(f_t) S_(t-1) + (1 - f_t) v_t^T, f_t = l + (1 - l) sigmoid(z_t) per key channel with a lower bound l; q = silu(.), no keys (HGRN2)
 //   matrix memory: S_t = exp(f + m_(t-1) - m_t) S_(t-1) + exp(i - m_t) k_t v_t^T with log gates i, f, a running maximum m and a normaliser n (xLSTM's mLSTM)
 enum HyLinearKind : int { HY_LIN_CHANNEL_DECAY = 0, HY_LIN_HEAD_DECAY = 1, HY_LIN_MATRIX_MEMORY = 2, HY_LIN_FORGET_WRITE = 3 };
-enum HyLinearNorm : int { HY_LIN_NORM_HEAD_WEIGHT = 0, HY_LIN_NORM_NONE = 1, HY_LIN_NORM_ALL_WEIGHT = 2 };   // weight of the per-head RMS norm: [vdim] shared by heads / none / [heads * vdim]
+enum HyLinearNorm : int { HY_LIN_NORM_HEAD_WEIGHT = 0, HY_LIN_NORM_NONE = 1, HY_LIN_NORM_ALL_WEIGHT = 2, HY_LIN_NORM_JOINT = 3 };   // weight of the per-head RMS norm: [vdim] shared by heads / none / [heads * vdim]; or one RMS norm over all heads together, weight [heads * vdim]
 
 struct HyLinear {
     int kind = HY_LIN_CHANNEL_DECAY, heads = 0, dim = 0, vdim = 0;
@@ -46,10 +50,11 @@ struct HyLinear {
     std::vector<float> decay;             // head decay: one per head
     int norm = HY_LIN_NORM_HEAD_WEIGHT, gate_silu = 1;      // output gate: silu (1) or sigmoid (0) of a projection, per channel (forget write: no output gate)
     bool q_scaled = true, k_scaled = false;                  // dim^-1/2 on q, or on k (after the rotation)
+    bool qkv_silu = false;                                   // the projections of q, k and v pass a SiLU
 };
 // down(silu(gate x) * up x) / down(relu(up x)^2) / down(gelu_tanh(up x)) / down(g sigmoid(slope g) (u + 1)) with g = min(gate x, limit), u = clamp(up x, -limit, limit) /
-// down(a N(z) + b N(z^2) + c N(z^3) + e) with z = up x and N(.) = unit RMS over the width (PolyNorm)
-enum HyExpertAct : int { HY_EXPERT_SWIGLU = 0, HY_EXPERT_RELU2 = 1, HY_EXPERT_GELU_TANH = 2, HY_EXPERT_CLAMPED_GLU = 3, HY_EXPERT_POLY_NORM = 4 };
+// down(a N(z) + b N(z^2) + c N(z^3) + e) with z = up x and N(.) = unit RMS over the width (PolyNorm) / down(gelu_tanh(gate x) * up x)
+enum HyExpertAct : int { HY_EXPERT_SWIGLU = 0, HY_EXPERT_RELU2 = 1, HY_EXPERT_GELU_TANH = 2, HY_EXPERT_CLAMPED_GLU = 3, HY_EXPERT_POLY_NORM = 4, HY_EXPERT_GELU_GLU = 5 };
 constexpr float HY_CLAMPED_GLU_SLOPE = 1.702f;
 enum HyRotLayout : int { HY_ROT_INTERLEAVED = 0, HY_ROT_HALVES = 1 };                         // channel 2i pairs with 2i + 1 / channel i with i + dims / 2
 // YaRN: with where(t) = dims ln(original / (2 pi t)) / (2 ln base), lo = max(floor(where(fast)), 0), hi = min(ceil(where(slow)), dims - 1) and
@@ -71,7 +76,8 @@ struct HyMoe {
 struct HyLayer {
     int type = HY_LATENT_ATTENTION;
     // latent attention: heads x (dim unrotated + rot_dim rotated) query/key, vdim values, kv_rank latent; rotary on the first rot_dims of the rotated part
-    // channel delta:    heads value heads of vdim, kv_heads query/key heads of dim, conv taps
+    // channel delta:    heads value heads of vdim, kv_heads query/key heads of dim, conv taps; head_decay: one decay per head and a full-rank SiLU gate
+    //                   instead of a decay per key channel and a low-rank sigmoid gate
     // mamba2:           heads x vdim inner channels, state N, groups of B/C, norm_groups, conv taps
     int heads = 0, kv_heads = 0, dim = 0, rot_dim = 0, vdim = 0, kv_rank = 0, rot_dims = 0, conv = 0, state = 0, groups = 1, norm_groups = 1;
     float rot_base = 10000.f, scale = 1.f;
@@ -85,7 +91,7 @@ struct HyLayer {
     int maps = 1, window = 0, keep_first = 0, qk_norm = 0, bias = 0, sink = 0, gate = HY_GATE_NONE, kv_from = -1;
     float diff = 0.f, softcap = 0.f, slope_exp = 0.f, q_temp_coef = 0.f; int q_temp_every = 0, out_bias = 0;
     // latent attention, optional parts: q_rank > 0: queries through a latent, q = W_uq rms_norm(W_dq h); rot_layout / rot_scaling: pairing and
-    // YaRN scaling of the rotary; window > 0: position i sees j with 0 <= i - j < window; sink; gate = HY_GATE_CHANNEL: sigmoid(W_g h) per channel.
+    // YaRN scaling of the rotary; window > 0: position i sees j with 0 <= i - j < window; sink; gate: sigmoid(W_g h) per channel or per head.
     // windowed attention, optional parts: conv > 0: a short causal convolution (no bias, no activation) on every channel of q, k and v, right
     // after the projection; rot_dims > 0: rotary on the first rot_dims channels of every query / key head; v_rot: the value of position j is
     // cached turned by j over all vdim channels (pair m by j rot_base^(-2m / vdim)), a head's output at position i is turned back by -i
@@ -93,7 +99,10 @@ struct HyLayer {
     // each, then a logarithmic scale up to bias_max, the last row beyond.  v_norm: a value head is cached divided by its RMS.  v_mix: every
     // such layer but the first caches (1 - lambda) v + lambda v_first, v_first = the first such layer's cached value of the same token (v_first: its layer, -1: this is the first)
     int bias_max = 0, v_norm = 0, v_mix = 0, v_first = -1;
-    int q_rank = 0, rot_layout = HY_ROT_INTERLEAVED, v_rot = 0;
+    int q_rank = 0, rot_layout = HY_ROT_INTERLEAVED, v_rot = 0, head_decay = 0;
+    // attention beside a linear recurrence (HY_ATTENTION_BESIDE_MEMORY): scaled_sum: the two outputs are joined as left_scale * left + right_scale * right
+    // instead of the halves of their RMS norms; rot_dims > 0: rotary on the attention side's queries and keys, after their norm
+    bool scaled_sum = false; float left_scale = 1.f, right_scale = 1.f;
     HyRotScaling rot_scaling;
     HyLinear lin;                         // HY_LINEAR_ATTENTION, and the memory side of HY_ATTENTION_BESIDE_MEMORY (whose attention side uses the fields above)
     HyMoe moe;
@@ -120,6 +129,8 @@ struct HybridConfig {
     // norm_around_zero: the layers' and the final norm weights are stored as w - 1
     bool branch_norm = false, norm_around_zero = false; float residual_mult = 1.f;
     bool loop_reinject = true;                          // a looped block re-injects the embedding before every pass (x <- W_in [x ; x0] + step[pass])
+    bool loop_add = false;                              // ... or adds it: before every pass but the first x <- x + x0, before every pass x <- x + step[pass]
+    bool single_stream = false;                         // sequential designs: one residual, sublayers' outputs join it as they are
     std::vector<HyLayer> layers;
     int loop_start = 0, loop_stop = 0, loop_times = 0;    // times == 0: no looped block
     std::vector<HyRun> runs;
@@ -156,6 +167,7 @@ struct HybridConfig {
         if (architecture == "Rofizen") return "rofizen";
         if (architecture == "Gosavik") return "gosavik";
         if (architecture == "Petipel") return "petipel";
+        if (architecture == "Ketopel") return "ketopel";
         return "";
     }
 
@@ -165,7 +177,8 @@ struct HybridConfig {
         HybridConfig c; c.dir = dir;
         c.arch = registry_key(j.str("architecture"));
         if (c.arch.empty()) throw std::runtime_error("config.json: unknown architecture '" + j.str("architecture") + "'");
-        const bool zu = c.arch == "zurevik", ro = c.arch == "rofizen", go = c.arch == "gosavik", pe = c.arch == "petipel";
+        const bool zu = c.arch == "zurevik", ro = c.arch == "rofizen", go = c.arch == "gosavik", pe = c.arch == "petipel", ke = c.arch == "ketopel";
+        if (ke) { c.norm = HY_RMS_NORM; c.sequential = true; c.single_stream = true; c.loop_reinject = false; c.loop_add = true; }
         if (go) {
             c.norm = HY_RMS_NORM; c.sequential = true; c.token_shift = true; c.loop_reinject = false;
             if (j.get("streams") && j.get("streams")->t == Json::Num) { c.streams = integer(j, "streams", "the model"); if (c.streams < 1 || c.streams > 8) throw std::runtime_error("config.json: streams must be 1 .. 8"); }
@@ -183,6 +196,19 @@ struct HybridConfig {
         c.logit_scale = j.get("logit_scale") ? (float)num(j, "logit_scale", "the model") : 1.f;
         const Json* ls = j.get("layers");
         if (!ls || ls->t != Json::Arr || ls->a.empty()) throw std::runtime_error("config.json: 'layers' must be a non-empty list");
+        auto read_scaling = [](HyLayer& l, const Json& rot) {        // optional YaRN scaling of a rotary
+            const Json* sc = rot.get("scaling");
+            if (!sc || sc->t != Json::Obj) return;
+            l.rot_scaling.on = true; l.rot_scaling.factor = (float)num(*sc, "factor", "scaling"); l.rot_scaling.original = (float)num(*sc, "original", "scaling");
+            l.rot_scaling.fast = (float)num(*sc, "fast", "scaling"); l.rot_scaling.slow = (float)num(*sc, "slow", "scaling");
+            if (!(l.rot_scaling.factor > 0.f) || !(l.rot_scaling.original > 0.f) || !(l.rot_scaling.fast > 0.f) || !(l.rot_scaling.slow > 0.f) || !(l.rot_base > 1.f))
+                throw std::runtime_error("config.json: bad rotary scaling");
+        };
+        auto read_decay = [](HyLinear& n, const Json& m, const char* where) {        // a fixed decay per head
+            const Json* d = m.get("decay");
+            if (!d || d->t != Json::Arr || (int)d->a.size() != n.heads) throw std::runtime_error(std::string("config.json: ") + where + " needs a list 'decay' with one number per head");
+            for (const Json& x : d->a) { if (x.t != Json::Num) throw std::runtime_error("config.json: 'decay' holds numbers"); n.decay.push_back((float)x.n); }
+        };
         for (const Json& lj : ls->a) {
             HyLayer l; const std::string type = lj.str("type");
             const Json& m = obj(lj, "mixer", "a layer");
@@ -196,20 +222,41 @@ struct HybridConfig {
                 if (go) {
                     l.q_rank = integer(m, "q_rank", type.c_str()); l.rot_layout = HY_ROT_HALVES; l.sink = 1; l.gate = HY_GATE_CHANNEL;
                     if (const Json* mk = m.get("mask")) if (mk->t == Json::Obj) { l.window = integer(*mk, "size", "mask"); if (l.window < 1) throw std::runtime_error("config.json: mask.size must be at least 1"); }
-                    if (const Json* sc = r.get("scaling")) if (sc->t == Json::Obj) {
-                        l.rot_scaling.on = true; l.rot_scaling.factor = (float)num(*sc, "factor", "scaling"); l.rot_scaling.original = (float)num(*sc, "original", "scaling");
-                        l.rot_scaling.fast = (float)num(*sc, "fast", "scaling"); l.rot_scaling.slow = (float)num(*sc, "slow", "scaling");
-                        if (!(l.rot_scaling.factor > 0.f) || !(l.rot_scaling.original > 0.f) || !(l.rot_scaling.fast > 0.f) || !(l.rot_scaling.slow > 0.f) || !(l.rot_base > 1.f))
-                            throw std::runtime_error("config.json: bad rotary scaling");
-                    }
+                    read_scaling(l, r);
                     if (l.q_rank <= 0 || l.dim < 0 || l.rot_dim < 0 || l.dim + l.rot_dim <= 0 || l.kv_rank <= 0 || l.kv_rank > 1024) throw std::runtime_error("config.json: bad latent attention sizes");
                 }
-            } else if (type == "channel_delta") {
+                if (ke) {
+                    l.gate = HY_GATE_HEAD; read_scaling(l, r);
+                    if (l.dim < 0 || l.rot_dim < 0 || l.dim + l.rot_dim <= 0 || l.rot_dims < 0 || l.kv_rank <= 0 || l.kv_rank > 1024 || !(l.rot_base > 0.f)) throw std::runtime_error("config.json: bad latent attention sizes");
+                }
+            } else if (!ke && type == "channel_delta") {
                 l.type = HY_CHANNEL_DELTA;
                 l.heads = integer(m, "heads", type.c_str()); l.kv_heads = integer(m, "kv_heads", type.c_str()); l.dim = integer(m, "dim", type.c_str());
                 l.vdim = integer(m, "vdim", type.c_str()); l.conv = integer(m, "conv", type.c_str());
                 if (l.kv_heads <= 0 || l.heads % l.kv_heads) throw std::runtime_error("config.json: kv_heads must divide heads");
-            } else if (type == "mamba2") {
+            } else if (ke && type == "delta") {
+                l.type = HY_CHANNEL_DELTA; l.head_decay = 1;
+                l.heads = integer(m, "heads", type.c_str()); l.kv_heads = integer(m, "kv_heads", type.c_str()); l.dim = integer(m, "dim", type.c_str());
+                l.vdim = integer(m, "vdim", type.c_str()); l.conv = integer(m, "conv", type.c_str());
+                if (l.kv_heads <= 0 || l.heads % l.kv_heads || l.dim <= 0 || l.dim > 760) throw std::runtime_error("config.json: bad delta-rule sizes");
+            } else if (ke && type == "parallel") {
+                // causal capped attention (left) beside lightning attention (right), both reading the layer's normed input
+                l.type = HY_ATTENTION_BESIDE_MEMORY; l.scaled_sum = true;
+                const Json& a = obj(m, "left", "parallel"); const Json& b = obj(m, "right", "parallel");
+                l.heads = integer(a, "heads", "left"); l.kv_heads = integer(a, "kv_heads", "left"); l.dim = integer(a, "dim", "left"); l.vdim = integer(a, "vdim", "left");
+                l.scale = (float)num(a, "scale", "left"); l.window = 1 << 30; l.qk_norm = 2;
+                l.left_scale = (float)num(m, "left_scale", "parallel"); l.right_scale = (float)num(m, "right_scale", "parallel");
+                if (a.get("softcap") && a.get("softcap")->t == Json::Num) l.softcap = (float)num(a, "softcap", "left");          // absent or 0: scores are not capped
+                const Json& r = obj(a, "rot", "left");
+                l.rot_base = (float)num(r, "base", "rot"); l.rot_dims = integer(r, "dims", "rot"); l.rot_layout = HY_ROT_HALVES; read_scaling(l, r);
+                if (l.heads <= 0 || l.kv_heads <= 0 || l.heads % l.kv_heads || l.dim <= 0 || l.vdim > 256 || l.dim > 1024 || l.softcap < 0.f || l.rot_dims < 0 || l.rot_dims > l.dim || (l.rot_dims & 1) || !(l.rot_base > 0.f))
+                    throw std::runtime_error("config.json: bad attention sizes");
+                HyLinear& n = l.lin;
+                n.kind = HY_LIN_HEAD_DECAY; n.heads = integer(b, "heads", "right"); n.dim = integer(b, "dim", "right"); n.vdim = integer(b, "vdim", "right");
+                n.norm = HY_LIN_NORM_JOINT; n.gate_silu = 0; n.q_scaled = false; n.qkv_silu = true;
+                read_decay(n, b, "lightning attention");
+                if (n.heads <= 0 || n.dim <= 0 || n.dim > 760 || n.vdim <= 0) throw std::runtime_error("config.json: bad linear-attention sizes");
+            } else if (!ke && type == "mamba2") {
                 l.type = HY_MAMBA2;
                 l.heads = integer(m, "heads", type.c_str()); l.vdim = integer(m, "vdim", type.c_str()); l.state = integer(m, "state", type.c_str());
                 l.groups = integer(m, "groups", type.c_str()); l.norm_groups = integer(m, "norm_groups", type.c_str()); l.conv = integer(m, "conv", type.c_str());
@@ -243,7 +290,7 @@ struct HybridConfig {
                 n.heads = l.heads = integer(m, "heads", type.c_str()); n.dim = l.dim = integer(m, "dim", type.c_str()); n.vdim = l.vdim = integer(m, "vdim", type.c_str());
                 n.kind = HY_LIN_FORGET_WRITE; n.norm = HY_LIN_NORM_HEAD_WEIGHT; n.q_scaled = false;
                 if (n.dim <= 0 || n.dim > 768) throw std::runtime_error("config.json: bad linear-attention sizes");
-            } else if (!pe && (type == "attention" || type == "attention_2")) {
+            } else if (!pe && !ke && (type == "attention" || type == "attention_2")) {
                 // "attention": differential (two score maps), query/key norm, kept first tokens, gate per channel;
                 // "attention_2": one map, projection biases, a sink per head, gate per head, optionally another layer's keys and values
                 const bool diff = type == "attention";
@@ -269,9 +316,7 @@ struct HybridConfig {
                 if (type == "gla") { n.kind = HY_LIN_CHANNEL_DECAY; n.tau = (float)num(m, "tau", "gla"); n.norm = HY_LIN_NORM_HEAD_WEIGHT; if (!(n.tau > 0.f)) throw std::runtime_error("config.json: gla needs tau > 0"); }
                 else {
                     n.kind = HY_LIN_HEAD_DECAY; n.norm = HY_LIN_NORM_NONE; n.q_scaled = false; n.k_scaled = true;
-                    const Json* d = m.get("decay");
-                    if (!d || d->t != Json::Arr || (int)d->a.size() != n.heads) throw std::runtime_error("config.json: retention needs a list 'decay' with one number per head");
-                    for (const Json& x : d->a) { if (x.t != Json::Num) throw std::runtime_error("config.json: 'decay' holds numbers"); n.decay.push_back((float)x.n); }
+                    read_decay(n, m, "retention");
                     const Json& r = obj(m, "rot", "retention");
                     n.rot_base = (float)num(r, "base", "rot"); n.rot_dims = integer(r, "dims", "rot");
                     if (n.rot_dims < 0 || n.rot_dims > n.dim || (n.rot_dims & 1)) throw std::runtime_error("config.json: rot.dims must be even and <= dim");
@@ -295,12 +340,12 @@ struct HybridConfig {
             const bool recurrent = l.type == HY_CHANNEL_DELTA || l.type == HY_MAMBA2;
             if (l.heads <= 0 || l.vdim <= 0 || (recurrent && (l.conv < 1 || l.conv > 16))) throw std::runtime_error("config.json: bad mixer sizes");
             const Json* mj = lj.get("mlp");
-            if (mj && mj->t == Json::Obj && (ro || go || pe) && mj->str("kind") == "dense") {
-                l.moe.present = true; l.moe.dense = true; l.moe.act = pe ? HY_EXPERT_POLY_NORM : go ? HY_EXPERT_GELU_TANH : HY_EXPERT_RELU2; l.moe.experts = 1; l.moe.top = 1;
+            if (mj && mj->t == Json::Obj && (ro || go || pe || ke) && mj->str("kind") == "dense") {
+                l.moe.present = true; l.moe.dense = true; l.moe.act = ke ? HY_EXPERT_GELU_GLU : pe ? HY_EXPERT_POLY_NORM : go ? HY_EXPERT_GELU_TANH : HY_EXPERT_RELU2; l.moe.experts = 1; l.moe.top = 1;
                 l.moe.ff = integer(*mj, "ff", "mlp");
                 if (l.moe.ff <= 0) throw std::runtime_error("config.json: bad feed-forward width");
             } else if (mj && mj->t == Json::Obj) {
-                if (go || mj->str("kind") != "moe") throw std::runtime_error("config.json: unknown mlp kind '" + mj->str("kind") + "'");
+                if (go || ke || mj->str("kind") != "moe") throw std::runtime_error("config.json: unknown mlp kind '" + mj->str("kind") + "'");
                 const Json& r = obj(*mj, "router", "mlp");
                 l.moe.present = true; l.moe.ff = integer(obj(*mj, "expert", "mlp"), "ff", "expert");
                 l.moe.experts = integer(r, "experts", "router"); l.moe.top = integer(r, "top", "router");

@@ -14,13 +14,20 @@ namespace {
 
 using namespace hyk;
 
+__device__ __forceinline__ float gemm_act(const HyGemmAct& a, float v, int n) {
+    if (a.kind == 1) { v = fmaxf(v, 0.f); return v * v; }
+    if (a.kind == 2) return gelu_tanhf_(v);
+    if (a.kind == 3 && n >= a.col0 && n < a.col1) return siluf_(v);
+    return v;
+}
+
 // ---------------------------------------------------------------------------------------------------------------------------------
 // GEMM: 64 x 64 tile, 16-wide k slices, 256 threads x (4 x 4) outputs.  The k order of every output is fixed (0..K-1), so a row's result
 // does not depend on which other rows share its launch.
 // ---------------------------------------------------------------------------------------------------------------------------------
 template <typename TA, int MODE>
 __global__ void __launch_bounds__(256) hy_gemm_kernel(const TA* __restrict__ A, int lda, const TA* __restrict__ B, int ldb, void* Cv, int ldc, int M, int N, int K,
-                                                      const float* __restrict__ bias, float alpha, long long sA, long long sB, long long sC, int act) {
+                                                      const float* __restrict__ bias, float alpha, long long sA, long long sB, long long sC, HyGemmAct act) {
     HY_PDL();
     __shared__ float As[16][64 + 4], Bs[16][64 + 4];
     A += (long long)blockIdx.z * sA; B += (long long)blockIdx.z * sB;
@@ -55,8 +62,7 @@ __global__ void __launch_bounds__(256) hy_gemm_kernel(const TA* __restrict__ A, 
             const int n = n0 + tx * 4 + j;
             if (n >= N) continue;
             float v = acc[i][j] * alpha + (bias ? bias[n] : 0.f);
-            if (act == 1) { v = fmaxf(v, 0.f); v *= v; }
-            else if (act == 2) v = gelu_tanhf_(v);
+            v = gemm_act(act, v, n);
             const long long at = (long long)blockIdx.z * sC + (long long)m * ldc + n;
             if (MODE == HY_STORE) stf(reinterpret_cast<TA*>(Cv) + at, v);
             else if (MODE == HY_STORE_F32) reinterpret_cast<float*>(Cv)[at] = v;
@@ -71,7 +77,7 @@ __global__ void __launch_bounds__(256) hy_gemm_kernel(const TA* __restrict__ A, 
 // at these sizes and runs K / 16 barrier-separated slices on a few CTAs.
 template <int MODE>
 __global__ void __launch_bounds__(256) hy_gemm_fewrows_kernel(const __nv_bfloat16* __restrict__ A, int lda, const __nv_bfloat16* __restrict__ B, int ldb, void* Cv, int ldc, int M, int N,
-                                                              int K, const float* __restrict__ bias, float alpha, long long sA, long long sB, long long sC, int act) {
+                                                              int K, const float* __restrict__ bias, float alpha, long long sA, long long sB, long long sC, HyGemmAct act) {
     HY_PDL();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = blockIdx.x * 8 + warp;
     if (n >= N) return;
@@ -93,8 +99,7 @@ __global__ void __launch_bounds__(256) hy_gemm_fewrows_kernel(const __nv_bfloat1
         acc = warp_sum(acc);
         if (lane == 0) {
             float v = acc * alpha + (bias ? bias[n] : 0.f);
-            if (act == 1) { v = fmaxf(v, 0.f); v *= v; }
-            else if (act == 2) v = gelu_tanhf_(v);
+            v = gemm_act(act, v, n);
             const long long at = (long long)blockIdx.y * sC + (long long)m * ldc + n;
             if (MODE == HY_STORE) reinterpret_cast<__nv_bfloat16*>(Cv)[at] = __float2bfloat16_rn(v);
             else if (MODE == HY_STORE_F32) reinterpret_cast<float*>(Cv)[at] = v;
@@ -233,7 +238,7 @@ __global__ void __launch_bounds__(128) hy_mla_attention_kernel(HyLatentAttn a, c
 #pragma unroll
     for (int w = 0; w < 4; ++w) { f[w] = mm[w] == -INFINITY ? 0.f : expf(mm[w] - M); L += f[w] * ll[w]; }
     if (a.sink) L += expf(sk - M);
-    const float inv = 1.0f / L;
+    const float inv = (a.head_gate ? sigmoidf_(ldf(reinterpret_cast<const TA*>(a.head_gate) + (long long)t * a.ldg + h)) : 1.0f) / L;
     for (int c = threadIdx.x; c < R; c += blockDim.x) {
         float v = 0.f;
 #pragma unroll
@@ -383,7 +388,8 @@ __global__ void __launch_bounds__(128) hy_mla_attention_mma_kernel(HyLatentAttn 
             const float m = half ? m_hi : m_lo, s2 = a.sink[h] * 1.4426950408889634f, M = fmaxf(m, s2);
             up = m == -INFINITY ? 0.f : exp2f(m - M); l = l * up + exp2f(s2 - M);
         }
-        const float inv = l > 0.f ? up / l : 0.f;
+        float inv = l > 0.f ? up / l : 0.f;
+        if (a.head_gate) inv *= sigmoidf_(ldf(reinterpret_cast<const __nv_bfloat16*>(a.head_gate) + (long long)row * a.ldg + h));
         __nv_bfloat16* dst = lat_out + ((long long)row * H + h) * R + vbase + (lane & 3) * 2;
 #pragma unroll
         for (int nb = 0; nb < NVB; ++nb) *reinterpret_cast<uint32_t*>(dst + nb * 8) = pack_bf16x2(o[nb][half * 2] * inv, o[nb][half * 2 + 1] * inv);
@@ -392,7 +398,8 @@ __global__ void __launch_bounds__(128) hy_mla_attention_mma_kernel(HyLatentAttn 
 
 // joins the parts of a decoding row: out = sum_p 2^(m_p - M) O_p / sum_p 2^(m_p - M) l_p, parts in order
 __global__ void __launch_bounds__(128) hy_mla_merge_kernel(const int32_t* item_row, const int32_t* item_slot0, const int32_t* item_parts, const float* ws_o,
-                                                           const float* ws_ml, __nv_bfloat16* lat_out, int H, int R, const float* sink) {
+                                                           const float* ws_ml, __nv_bfloat16* lat_out, int H, int R, const float* sink,
+                                                           const __nv_bfloat16* head_gate, int ldg) {
     HY_PDL();
     const int row = item_row[blockIdx.x], slot0 = item_slot0[blockIdx.x], P = item_parts[blockIdx.x], h = blockIdx.y;
     const float s2 = sink ? sink[h] * 1.4426950408889634f : -INFINITY;       // the sink, in the partials' base-2 units
@@ -400,7 +407,7 @@ __global__ void __launch_bounds__(128) hy_mla_merge_kernel(const int32_t* item_r
     for (int p = 0; p < P; ++p) M = fmaxf(M, ws_ml[((long long)(slot0 + p) * H + h) * 2]);
     float L = sink ? exp2f(s2 - M) : 0.f;
     for (int p = 0; p < P; ++p) { const float* ml = ws_ml + ((long long)(slot0 + p) * H + h) * 2; L += exp2f(ml[0] - M) * ml[1]; }
-    const float inv = 1.0f / L;
+    const float inv = (head_gate ? sigmoidf_(ldf(head_gate + (long long)row * ldg + h)) : 1.0f) / L;
     for (int c = threadIdx.x; c < R; c += blockDim.x) {
         float acc = 0.f;
         for (int p = 0; p < P; ++p) acc += exp2f(ws_ml[((long long)(slot0 + p) * H + h) * 2] - M) * ws_o[((long long)(slot0 + p) * H + h) * R + c];
@@ -538,7 +545,8 @@ __global__ void __launch_bounds__(128) hy_mha_prefill_mma_kernel(HyLatentAttn a,
             const float m = half ? m_hi : m_lo, s2 = a.sink[h] * 1.4426950408889634f, M = fmaxf(m, s2);
             up = m == -INFINITY ? 0.f : exp2f(m - M); l = l * up + exp2f(s2 - M);
         }
-        const float inv = l > 0.f ? up / l : 0.f;
+        float inv = l > 0.f ? up / l : 0.f;
+        if (a.head_gate) inv *= sigmoidf_(ldf(reinterpret_cast<const __nv_bfloat16*>(a.head_gate) + (long long)(row0 + qi) * a.ldg + h));
         __nv_bfloat16* dst = mix + (long long)(row0 + qi) * ld_mix + h * VD + (lane & 3) * 2;
         const __nv_bfloat16* gp = a.gate ? reinterpret_cast<const __nv_bfloat16*>(a.gate) + (long long)(row0 + qi) * a.ldg + h * VD + (lane & 3) * 2 : nullptr;
 #pragma unroll
@@ -656,6 +664,7 @@ template <typename TA>
 __global__ void __launch_bounds__(128) hy_delta_prep_kernel(HyDelta d, const TA* conv, int ld_conv, const TA* b, int ld_b, const TA* a, int ld_a, const float* A_log,
                                                              const float* dt_bias, float* qq, float* kk, float* vv, float* dec, float* beta) {
     HY_PDL();
+    const int ND = d.head_decay ? 1 : d.dim;                    // decays per head
     const int t = blockIdx.x, KH = d.kv_heads, H = d.heads, D = d.dim, VD = d.vdim;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const TA* cr = conv + (long long)t * ld_conv;
@@ -670,8 +679,8 @@ __global__ void __launch_bounds__(128) hy_delta_prep_kernel(HyDelta d, const TA*
     }
     for (int i = threadIdx.x; i < H * VD; i += blockDim.x) vv[(long long)t * H * VD + i] = ldf(cr + 2 * KH * D + i);
     for (int i = threadIdx.x; i < H; i += blockDim.x) beta[(long long)t * H + i] = sigmoidf_(ldf(b + (long long)t * ld_b + i));
-    for (int i = threadIdx.x; i < H * D; i += blockDim.x)
-        dec[(long long)t * H * D + i] = expf(-expf(A_log[i / D]) * softplusf_(ldf(a + (long long)t * ld_a + i) + dt_bias[i]));
+    for (int i = threadIdx.x; i < H * ND; i += blockDim.x)
+        dec[(long long)t * H * ND + i] = expf(-expf(A_log[i / ND]) * softplusf_(ldf(a + (long long)t * ld_a + i) + dt_bias[i]));
 }
 template <typename TA>
 __global__ void __launch_bounds__(128) hy_mamba_prep_kernel(HyMamba m, const TA* conv, int ld_conv, const TA* dt, int ld_dt, const float* A_log, const float* dt_bias,
@@ -694,7 +703,7 @@ constexpr int REC_COLS = 64;      // state columns (value channels) per CTA; a c
 template <int MODE>
 __global__ void __launch_bounds__(REC_COLS) hy_recurrence_kernel(const float* qq, const float* kk, const float* vv, const float* dec, const float* beta, float* out,
                                                                  float* state, int H, int QH, int D, int VD, HyRows r, float* norm_state, float* norm_out) {
-    constexpr bool DELTA = MODE == HY_REC_DELTA, CH = MODE != HY_REC_SCALAR;
+    constexpr bool DELTA = MODE == HY_REC_DELTA || MODE == HY_REC_DELTA_HEAD, CH = MODE == HY_REC_DELTA || MODE == HY_REC_CHANNEL;      // CH: a decay per key channel
     HY_PDL();
     extern __shared__ float sm[];
     float* S = sm;                         // [D][REC_COLS]
@@ -716,8 +725,8 @@ __global__ void __launch_bounds__(REC_COLS) hy_recurrence_kernel(const float* qq
         const float v = is_norm ? 1.f : ok ? vv[(t * H + h) * VD + col] : 0.f;
         float o = 0.f;
         if (DELTA) {
-            float dot = 0.f;
-            for (int d = 0; d < D; ++d) { const float s = S[d * REC_COLS + j] * ds[d]; S[d * REC_COLS + j] = s; dot = fmaf(s, ks[d], dot); }
+            float dot = 0.f; const float a = CH ? 1.f : dec[t * H + h];
+            for (int d = 0; d < D; ++d) { const float s = S[d * REC_COLS + j] * (CH ? ds[d] : a); S[d * REC_COLS + j] = s; dot = fmaf(s, ks[d], dot); }
             const float u = beta[t * H + h] * (v - dot);
             for (int d = 0; d < D; ++d) { const float s = fmaf(ks[d], u, S[d * REC_COLS + j]); S[d * REC_COLS + j] = s; o = fmaf(s, qs[d], o); }
         } else if (CH) {
@@ -746,7 +755,7 @@ __global__ void __launch_bounds__(128) hy_recurrence_reg_kernel(const float* __r
                                                                 const float* __restrict__ dec, const float* __restrict__ beta, float* __restrict__ out,
                                                                 float* __restrict__ state, int H, int QH, int D, int VD, HyRows r, float* __restrict__ norm_state,
                                                                 float* __restrict__ norm_out) {
-    constexpr bool DELTA = MODE == HY_REC_DELTA, CH = MODE != HY_REC_SCALAR;
+    constexpr bool DELTA = MODE == HY_REC_DELTA || MODE == HY_REC_DELTA_HEAD, CH = MODE == HY_REC_DELTA || MODE == HY_REC_CHANNEL;      // CH: a decay per key channel
     HY_PDL();
     extern __shared__ __align__(16) float rec_ring[];
     constexpr int stride = 3 * DM + REC_CTA_COLS + 4;     // floats per stage: q[DM] k[DM] g[DM] v[128] scalar (padded to 16 bytes); pad rows: q = k = 0, decay 1
@@ -774,13 +783,13 @@ __global__ void __launch_bounds__(128) hy_recurrence_reg_kernel(const float* __r
         const int c = tid - 96;
         if (c * 4 < COLS && blockIdx.z * COLS + c * 4 < VD) { src = vv + ((long long)row0 * H + h) * VD + blockIdx.z * COLS + c * 4; step = (long long)H * VD; dst = 3 * DM + c * 4; }
     }
-    const float* src_sc = (tid == 0 && MODE != HY_REC_CHANNEL) ? (DELTA ? beta : dec) + (long long)row0 * H + h : nullptr;
+    const float* src_sc = (tid == 0 && MODE != HY_REC_CHANNEL) ? (DELTA ? beta : dec) + (long long)row0 * H + h : (tid == 1 && MODE == HY_REC_DELTA_HEAD) ? dec + (long long)row0 * H + h : nullptr;
     int issued = 0;
     auto issue = [&]() {                             // next token of the sequence's rows -> ring slot issued % REC_STAGES
         if (issued < len) {
             float* slot = rec_ring + (issued % REC_STAGES) * stride;
             if (src) { cp_async16(slot + dst, src); src += step; }
-            if (src_sc) { asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(slot + 3 * DM + REC_CTA_COLS)), "l"(src_sc) : "memory"); src_sc += H; }
+            if (src_sc) { asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(slot + 3 * DM + REC_CTA_COLS + tid)), "l"(src_sc) : "memory"); src_sc += H; }
         }
         ++issued;
         asm volatile("cp.async.commit_group;" ::: "memory");
@@ -797,14 +806,14 @@ __global__ void __launch_bounds__(128) hy_recurrence_reg_kernel(const float* __r
         issue();
         if (LANES == 4 && i > 0) join(i - 1);        // its partials were written before this barrier; their buffer is written again at token i + 1, behind the next one
         const float* slot = rec_ring + (i % REC_STAGES) * stride;
-        const float v = is_norm ? 1.f : slot[3 * DM + cl], sc = slot[3 * DM + REC_CTA_COLS];
+        const float v = is_norm ? 1.f : slot[3 * DM + cl], sc = slot[3 * DM + REC_CTA_COLS], gh = MODE == HY_REC_DELTA_HEAD ? slot[3 * DM + REC_CTA_COLS + 1] : 1.f;
         const float* sq = slot + r0; const float* sk = slot + DM + r0; const float* sg = slot + 2 * DM + r0;
         float o0 = 0.f, o1 = 0.f, o2 = 0.f, o3 = 0.f;
         if (DELTA) {
             float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;
 #pragma unroll
             for (int j = 0; j < DR; j += 4) {
-                const float4 g4 = *reinterpret_cast<const float4*>(sg + j), k4 = *reinterpret_cast<const float4*>(sk + j);
+                const float4 g4 = CH ? *reinterpret_cast<const float4*>(sg + j) : make_float4(gh, gh, gh, gh), k4 = *reinterpret_cast<const float4*>(sk + j);
                 S[j] *= g4.x; S[j + 1] *= g4.y; S[j + 2] *= g4.z; S[j + 3] *= g4.w;
                 d0 = fmaf(S[j], k4.x, d0); d1 = fmaf(S[j + 1], k4.y, d1); d2 = fmaf(S[j + 2], k4.z, d2); d3 = fmaf(S[j + 3], k4.w, d3);
             }
@@ -1183,6 +1192,15 @@ __global__ void __launch_bounds__(256) hy_argmax_rows_kernel(float* logits, int 
         out_ids[blockIdx.x] = i < V ? i : 0;
     }
 }
+// gate / up products side by side in blocks of 16 -> gelu_tanh(gate) * up
+template <typename TA>
+__global__ void hy_gelu_glu_kernel(const TA* __restrict__ gu, int ld, TA* __restrict__ out, int ldo, int ff) {
+    HY_PDL();
+    const long long t = blockIdx.y; const int f = blockIdx.x * blockDim.x + threadIdx.x;
+    if (f >= ff) return;
+    const TA* p = gu + t * ld + (f >> 4) * 32 + (f & 15);
+    stf(out + t * ldo + f, gelu_tanhf_(ldf(p)) * ldf(p + 16));
+}
 __global__ void hy_add_rowvec_kernel(float* x, const float* v, int W) {
     HY_PDL();
     for (int c = threadIdx.x; c < W; c += blockDim.x) x[(long long)blockIdx.x * W + c] += v[c];
@@ -1195,7 +1213,7 @@ using bf = __nv_bfloat16;
 
 template <typename TA>
 static cudaError_t gemm_t(int mode, const void* A, int lda, const void* B, int ldb, void* C, int ldc, int M, int N, int K, const float* bias, float alpha, int batch,
-                          long long sA, long long sB, long long sC, cudaStream_t s, int act) {
+                          long long sA, long long sB, long long sC, cudaStream_t s, HyGemmAct act) {
     dim3 grid((N + 63) / 64, (M + 63) / 64, batch);
     const TA* a = reinterpret_cast<const TA*>(A); const TA* b = reinterpret_cast<const TA*>(B);
     switch (mode) {
@@ -1206,7 +1224,7 @@ static cudaError_t gemm_t(int mode, const void* A, int lda, const void* B, int l
     return cudaErrorInvalidValue;
 }
 cudaError_t hy_gemm(bool f32, int mode, const void* A, int lda, const void* B, int ldb, void* C, int ldc, int M, int N, int K, const float* bias, float alpha, int batch,
-                    long long sA, long long sB, long long sC, cudaStream_t s, int act) {
+                    long long sA, long long sB, long long sC, cudaStream_t s, HyGemmAct act) {
     if (M <= 0 || N <= 0 || K <= 0 || batch <= 0) return cudaSuccess;
     auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
     if (!f32 && M <= HY_GEMM_FEW_ROWS && K % 8 == 0 && K <= 1024 && lda % 8 == 0 && ldb % 8 == 0 && sA % 8 == 0 && sB % 8 == 0 && al16(A) && al16(B)) {
@@ -1266,9 +1284,9 @@ static cudaError_t mla_mma_launch(const HyLatentAttn& a, const float* q_abs, con
                         tile_seq, tile_q0, sp);
 }
 cudaError_t hy_mla_merge(const int32_t* item_row, const int32_t* item_slot0, const int32_t* item_parts, int n_items, const float* ws_o, const float* ws_ml, void* lat_out,
-                         int heads, int kv_rank, cudaStream_t s, const float* sink) {
+                         int heads, int kv_rank, cudaStream_t s, const float* sink, const void* head_gate, int ldg) {
     if (n_items <= 0) return cudaSuccess;
-    return launch_plain(hy_mla_merge_kernel, dim3(n_items, heads), dim3(128), 0, s, item_row, item_slot0, item_parts, ws_o, ws_ml, (bf*)lat_out, heads, kv_rank, sink);
+    return launch_plain(hy_mla_merge_kernel, dim3(n_items, heads), dim3(128), 0, s, item_row, item_slot0, item_parts, ws_o, ws_ml, (bf*)lat_out, heads, kv_rank, sink, (const bf*)head_gate, ldg);
 }
 cudaError_t hy_mla_attention_mma(const HyLatentAttn& a, const float* q_abs, const void* cache, void* lat_out, const HyRows& r, const int32_t* tile_seq,
                                  const int32_t* tile_q0, int n_tiles, const HyMlaSplit& sp, cudaStream_t s) {
@@ -1285,7 +1303,7 @@ cudaError_t hy_mla_attention_mma(const HyLatentAttn& a, const float* q_abs, cons
 }
 static int mha_nvb(const HyLatentAttn& a) {
     if ((a.dim + a.rot_dim) % 16 != 0 || a.dim % 8 != 0 || a.rot_dim % 8 != 0 || a.kv_rank % 8 != 0) return 0;
-    return a.vdim == 128 ? 16 : a.vdim == 64 ? 8 : a.vdim == 32 ? 4 : a.vdim == 16 ? 2 : 0;
+    return a.vdim % 16 == 0 && a.vdim >= 16 && a.vdim <= 128 ? a.vdim / 8 : 0;
 }
 bool hy_mha_prefill_supported(const HyLatentAttn& a) { return mha_nvb(a) != 0 && a.dim + a.rot_dim <= 512; }
 cudaError_t hy_gather_ctx(const void* cache, int E, const HyRows& r, const int32_t* seq_base, int max_ctx, void* lat_ctx, cudaStream_t s) {
@@ -1307,7 +1325,11 @@ cudaError_t hy_mha_prefill(const HyLatentAttn& a, const void* q, int ldq, const 
     if (n_tiles <= 0) return cudaSuccess;
     switch (mha_nvb(a)) {
         case 16: return mha_launch<16>(a, q, ldq, q_abs, kv_ctx, ld_kv, lat_ctx, mix, ld_mix, r, tile_seq, tile_head, tile_row0, seq_base, n_tiles, s);
+        case 14: return mha_launch<14>(a, q, ldq, q_abs, kv_ctx, ld_kv, lat_ctx, mix, ld_mix, r, tile_seq, tile_head, tile_row0, seq_base, n_tiles, s);
+        case 12: return mha_launch<12>(a, q, ldq, q_abs, kv_ctx, ld_kv, lat_ctx, mix, ld_mix, r, tile_seq, tile_head, tile_row0, seq_base, n_tiles, s);
+        case 10: return mha_launch<10>(a, q, ldq, q_abs, kv_ctx, ld_kv, lat_ctx, mix, ld_mix, r, tile_seq, tile_head, tile_row0, seq_base, n_tiles, s);
         case 8: return mha_launch<8>(a, q, ldq, q_abs, kv_ctx, ld_kv, lat_ctx, mix, ld_mix, r, tile_seq, tile_head, tile_row0, seq_base, n_tiles, s);
+        case 6: return mha_launch<6>(a, q, ldq, q_abs, kv_ctx, ld_kv, lat_ctx, mix, ld_mix, r, tile_seq, tile_head, tile_row0, seq_base, n_tiles, s);
         case 4: return mha_launch<4>(a, q, ldq, q_abs, kv_ctx, ld_kv, lat_ctx, mix, ld_mix, r, tile_seq, tile_head, tile_row0, seq_base, n_tiles, s);
         case 2: return mha_launch<2>(a, q, ldq, q_abs, kv_ctx, ld_kv, lat_ctx, mix, ld_mix, r, tile_seq, tile_head, tile_row0, seq_base, n_tiles, s);
     }
@@ -1346,7 +1368,7 @@ cudaError_t hy_mamba_prep(bool f32, const HyMamba& m, const void* conv, int ld_c
 }
 cudaError_t hy_recurrence(int mode, const float* qq, const float* kk, const float* vv, const float* dec, const float* beta, float* out, float* state, int heads,
                           int qk_heads, int dim, int vdim, const HyRows& r, cudaStream_t s, float* norm_state, float* norm_out) {
-    if (mode < 0 || mode > 2 || (norm_state && (mode == HY_REC_DELTA || !norm_out))) return cudaErrorInvalidValue;
+    if (mode < 0 || mode > HY_REC_DELTA_HEAD || (norm_state && (mode == HY_REC_DELTA || mode == HY_REC_DELTA_HEAD || !norm_out))) return cudaErrorInvalidValue;
     const int cols = vdim + (norm_state ? 1 : 0);
     if (dim <= 128 && dim % 4 == 0 && vdim % 4 == 0) {
         // one thread per column runs a chain of 4 dim dependent-ish operations per token with one or two warps per scheduler; beyond 32
@@ -1358,6 +1380,7 @@ cudaError_t hy_recurrence(int mode, const float* qq, const float* kk, const floa
 #define HY_REC(MD, DM, LN) launch_plain(hy_recurrence_reg_kernel<MD, DM, LN>, grid, dim3(128), ring, s, qq, kk, vv, dec, beta, out, state, heads, qk_heads, dim, vdim, r, norm_state, norm_out)
 #define HY_REC_DM(MD, LN) (dm == 32 ? HY_REC(MD, 32, LN) : dm == 64 ? HY_REC(MD, 64, LN) : HY_REC(MD, 128, LN))
         if (mode == HY_REC_DELTA) return wide ? HY_REC_DM(HY_REC_DELTA, 4) : HY_REC_DM(HY_REC_DELTA, 1);
+        if (mode == HY_REC_DELTA_HEAD) return wide ? HY_REC_DM(HY_REC_DELTA_HEAD, 4) : HY_REC_DM(HY_REC_DELTA_HEAD, 1);
         if (mode == HY_REC_CHANNEL) return wide ? HY_REC_DM(HY_REC_CHANNEL, 4) : HY_REC_DM(HY_REC_CHANNEL, 1);
         return wide ? HY_REC_DM(HY_REC_SCALAR, 4) : HY_REC_DM(HY_REC_SCALAR, 1);
 #undef HY_REC_DM
@@ -1365,16 +1388,17 @@ cudaError_t hy_recurrence(int mode, const float* qq, const float* kk, const floa
     }
     const size_t smem = (size_t)(dim * REC_COLS + 3 * dim) * 4;
     dim3 grid(r.S, heads, (cols + REC_COLS - 1) / REC_COLS);
-    static bool attr_done[3][16] = {};
+    static bool attr_done[4][16] = {};
     if (smem > 200 * 1024) return cudaErrorInvalidValue;
     if (smem > 48 * 1024) {      // the limit is set once per kernel and device: raise it to the most any size may ask for
         cudaError_t e = mode == HY_REC_DELTA ? ensure_dynamic_smem(hy_recurrence_kernel<HY_REC_DELTA>, 200 * 1024, attr_done[0])
+                      : mode == HY_REC_DELTA_HEAD ? ensure_dynamic_smem(hy_recurrence_kernel<HY_REC_DELTA_HEAD>, 200 * 1024, attr_done[3])
                       : mode == HY_REC_CHANNEL ? ensure_dynamic_smem(hy_recurrence_kernel<HY_REC_CHANNEL>, 200 * 1024, attr_done[2])
                                                : ensure_dynamic_smem(hy_recurrence_kernel<HY_REC_SCALAR>, 200 * 1024, attr_done[1]);
         if (e != cudaSuccess) return e;
     }
 #define HY_RECG(MD) launch_plain(hy_recurrence_kernel<MD>, grid, dim3(REC_COLS), smem, s, qq, kk, vv, dec, beta, out, state, heads, qk_heads, dim, vdim, r, norm_state, norm_out)
-    return mode == HY_REC_DELTA ? HY_RECG(HY_REC_DELTA) : mode == HY_REC_CHANNEL ? HY_RECG(HY_REC_CHANNEL) : HY_RECG(HY_REC_SCALAR);
+    return mode == HY_REC_DELTA ? HY_RECG(HY_REC_DELTA) : mode == HY_REC_DELTA_HEAD ? HY_RECG(HY_REC_DELTA_HEAD) : mode == HY_REC_CHANNEL ? HY_RECG(HY_REC_CHANNEL) : HY_RECG(HY_REC_SCALAR);
 #undef HY_RECG
 }
 cudaError_t hy_gated_norm(bool f32, const float* o, int C, int group, const float* w, int wlen, const void* gate, int ld_gate, int gate_before, int act, const float* skip,
@@ -1438,6 +1462,11 @@ cudaError_t hy_gather_rows_f32(const float* x, const int32_t* rows, float* out, 
 cudaError_t hy_argmax_rows(float* logits, int n, int V, float softcap, int32_t* out_ids, cudaStream_t s) {
     if (n <= 0) return cudaSuccess;
     return launch_plain(hy_argmax_rows_kernel, dim3(n), dim3(256), 0, s, logits, V, softcap, out_ids);
+}
+cudaError_t hy_gelu_glu(bool f32, const void* gu, int ld, void* out, int ldo, int ff, int T, cudaStream_t s) {
+    const dim3 grid((ff + 255) / 256, T);
+    return f32 ? launch_plain(hy_gelu_glu_kernel<float>, grid, dim3(256), 0, s, (const float*)gu, ld, (float*)out, ldo, ff)
+               : launch_plain(hy_gelu_glu_kernel<bf>, grid, dim3(256), 0, s, (const bf*)gu, ld, (bf*)out, ldo, ff);
 }
 cudaError_t hy_add_rowvec(float* x, const float* v, int T, int W, cudaStream_t s) { return launch_plain(hy_add_rowvec_kernel, dim3(T), dim3(256), 0, s, x, v, W); }
 

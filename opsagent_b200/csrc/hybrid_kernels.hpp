@@ -35,11 +35,12 @@ struct HyRows {
 enum HyGemmMode : int { HY_STORE = 0, HY_STORE_F32 = 1, HY_ACC_F32 = 2 };
 // C[z][M,N] (op)= alpha * A[z][M,K] . B[z][N,K]^T (+ bias[N]), z < batch with element strides sA/sB/sC.  Plain tiled FMA GEMM in fp32
 // accumulation for any sizes: the fp32 mode's matrix product, and the bf16 mode's fallback where a shape does not fit the tensor-core tiles.
-// act = 1: the stored value is relu(.)^2, act = 2: the tanh form of GELU (HY_STORE / HY_STORE_F32)
+// act.kind = 1: the stored value is relu(.)^2, 2: the tanh form of GELU, 3: SiLU on columns col0 .. col1 - 1 (HY_STORE / HY_STORE_F32)
+struct HyGemmAct { int kind = 0, col0 = 0, col1 = 0; };
 // bf16 steps of at most HY_GEMM_FEW_ROWS rows with K <= 1024 in aligned groups of 8 take a one-warp-per-output-column kernel instead of the tile kernel
 constexpr int HY_GEMM_FEW_ROWS = 32;
 cudaError_t hy_gemm(bool f32, int mode, const void* A, int lda, const void* B, int ldb, void* C, int ldc, int M, int N, int K, const float* bias,
-                    float alpha, int batch, long long sA, long long sB, long long sC, cudaStream_t s, int act = 0);
+                    float alpha, int batch, long long sA, long long sB, long long sC, cudaStream_t s, HyGemmAct act = HyGemmAct());
 
 // x[t] = table[ids[t]] * scale (fp32); x0 (optional) keeps a copy for a looped block's re-injection
 // h (optional, [T, ldh] in the activation type): the same rows as the input of sublayers that read the residual itself
@@ -95,8 +96,9 @@ bool hy_win_supported(const HyWinAttn& a);
 // q [T, ldq] (head by head, map by map): RMS-normed in place with q_norm_w when qk_norm; k / v [T, ldkv] (null: this layer reads a cache
 // another layer fills): keys normed alike with k_norm_w, both stored at cache row slots[t].  qk_norm = 2: one norm over the row's whole q (k) projection,
 // weights of that size, then the query temperature
+// — and, where rot is given, the rotary of the first rot->dims channels of every query and key head (no value rotation)
 cudaError_t hy_win_prep(bool f32, const HyWinAttn& a, void* q, int ldq, const void* k, const void* v, int ldkv, const float* q_norm_w, const float* k_norm_w, float eps, void* cache,
-                        const HyRows& r, cudaStream_t s);
+                        const HyRows& r, cudaStream_t s, const HyRotary* rot = nullptr);
 // plain form (any sizes, both element types; prefill rows and decoding rows alike): out[t, head * vdim ..] in the activation type
 cudaError_t hy_win_attention(bool f32, const HyWinAttn& a, const void* q, int ldq, const void* cache, const float* sink, const void* gate, int ldg, void* out, int ldo, float eps,
                              const HyRows& r, cudaStream_t s);
@@ -122,6 +124,8 @@ struct HyLatentAttn {             // sizes of one latent-attention layer
     int window = 0, rot_layout = 0; const float* sink = nullptr;
     // prefill form only: out[t, c] *= sigmoid(gate[t, c]) over the concatenated heads (bf16, pitch ldg), in the attention kernel's epilogue
     const void* gate = nullptr; int ldg = 0;
+    // every form: head h's output in row t is multiplied by sigmoid(head_gate[t, h]) (activation type, pitch ldg); the absorbed forms scale the latent read-out
+    const void* head_gate = nullptr;
 };
 // From the q projection (q: [T, ldq], head by head [dim | rot_dim]) and the down projection (ckv: [T, ldc] = [kv_rank | rot_dim]):
 // latent = rmsnorm(ckv[:rank]) * norm_w and the rotated shared key go to cache row slots[t] ([rank + rot_dim] per row); the rotated query
@@ -143,9 +147,9 @@ bool hy_mla_mma_supported(const HyLatentAttn& a);
 cudaError_t hy_mla_attention_mma(const HyLatentAttn& a, const float* q_abs, const void* cache, void* lat_out, const HyRows& r, const int32_t* tile_seq,
                                  const int32_t* tile_q0, int n_tiles, const HyMlaSplit& sp, cudaStream_t s);
 cudaError_t hy_mla_merge(const int32_t* item_row, const int32_t* item_slot0, const int32_t* item_parts, int n_items, const float* ws_o, const float* ws_ml, void* lat_out,
-                         int heads, int kv_rank, cudaStream_t s, const float* sink = nullptr);
+                         int heads, int kv_rank, cudaStream_t s, const float* sink = nullptr, const void* head_gate = nullptr, int ldg = 0);
 
-// Prefill form (bf16; dim and rot_dim multiples of 8, their sum of 16, vdim 16 / 32 / 64 / 128): hy_gather_ctx copies the cache rows 0..ctx-1 of
+// Prefill form (bf16; dim and rot_dim multiples of 8, their sum of 16, vdim a multiple of 16 up to 128): hy_gather_ctx copies the cache rows 0..ctx-1 of
 // the sequences with seq_base[s] >= 0 to lat_ctx[seq_base[s] + j]; a GEMM makes kv_ctx = lat_ctx[:, :rank] . [W_uk ; W_uv]^T ([rows, heads dim |
 // heads vdim]); hy_mha_prefill then runs causal attention per (sequence, head) — a tile is 64 query rows starting at row tile_row0 of its
 // sequence — and writes mix[row, head * vdim ..].  Queries: unrotated part from q ([T, ldq], head by head [dim | rot_dim]), rotated part
@@ -162,8 +166,9 @@ cudaError_t hy_conv_silu(bool f32, const void* in, int ld_in, int C, const float
                          const void* tails, const HyRows& r, cudaStream_t s, int act = 1);
 cudaError_t hy_conv_tails(bool f32, const void* in, int ld_in, int C, int taps, void* tails, const HyRows& r, cudaStream_t s);
 
-struct HyDelta { int heads, kv_heads, dim, vdim; };
-// unit-norm q (times dim^-1/2) and k, v, beta = sigmoid(b), per-channel decay exp(-exp(A_log_h) softplus(a + dt_bias)) — all fp32
+struct HyDelta { int heads, kv_heads, dim, vdim, head_decay = 0; };
+// unit-norm q (times dim^-1/2) and k, v, beta = sigmoid(b), decay exp(-exp(A_log_h) softplus(a + dt_bias)) per key channel (a, dt_bias, dec: [heads, dim])
+// or, head_decay, per head (a, dt_bias, dec: [heads]) — all fp32
 cudaError_t hy_delta_prep(bool f32, const HyDelta& d, const void* qkv_conv, int ld_conv, const void* b, int ld_b, const void* a, int ld_a,
                           const float* A_log, const float* dt_bias, float* qq, float* kk, float* vv, float* dec, float* beta, int T, cudaStream_t s);
 struct HyMamba { int heads, vdim, state, groups; };
@@ -173,11 +178,12 @@ cudaError_t hy_mamba_prep(bool f32, const HyMamba& m, const void* xbc_conv, int 
 // The linear recurrence both mixers share, per (sequence, head) on an fp32 state S[dim, vdim] carried in `state` (slot-major):
 //   delta:  S <- diag(dec_t) S;  u = beta_t (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t
 //   plain:  S <- dec_t S + k_t v_t^T;                                            o_t = S^T q_t
+//   delta, one decay per head (dec [T, heads]): the delta form with dec_t a number
 // qq/kk: [T, qk_heads, dim]; vv/out: [T, heads, vdim]; dec: [T, heads, dim] (delta) or [T, heads]; head h reads q/k head h / (heads / qk_heads)
 // mode HY_REC_CHANNEL: S <- diag(dec_t) S + k_t v_t^T with dec [T, heads, dim] (gated linear attention).
 // norm_state != null (plain modes): one more value channel whose value is always 1 — the normaliser n_t = dec_t n_(t-1) + k_t, kept in
 // norm_state [slots, heads, dim]; its read-out n_t . q_t goes to norm_out [T, heads].
-enum HyRecMode : int { HY_REC_SCALAR = 0, HY_REC_DELTA = 1, HY_REC_CHANNEL = 2 };
+enum HyRecMode : int { HY_REC_SCALAR = 0, HY_REC_DELTA = 1, HY_REC_CHANNEL = 2, HY_REC_DELTA_HEAD = 3 };
 cudaError_t hy_recurrence(int mode, const float* qq, const float* kk, const float* vv, const float* dec, const float* beta, float* out,
                           float* state, int heads, int qk_heads, int dim, int vdim, const HyRows& r, cudaStream_t s, float* norm_state = nullptr, float* norm_out = nullptr);
 
@@ -264,7 +270,9 @@ cudaError_t hy_poly_norm(bool f32, void* z, int ldz, int n, const HyPolyCoef& k,
 //      choices (in order) of b.y[b.dst_of[t * top + c]] (grouped experts: the rows of their sorted tiles)
 //  (2) w != null: h[t] = x / sqrt(mean(x^2) + eps) * w of the new x (activation type, pitch ldh).  rows != null: output row t reads row rows[t] of x
 //      and y, and x itself stays
-struct HyBranch { const float* y; const float* w; float mult; const int32_t* dst_of; int top; };
+// b.w == null: y joins as it is, x[t] <- x[t] + b.mult * y.  Between (1) and (2), each optional: x[t] += b.add_rows[t] ([T, W]), then x[t] += b.add_vec ([W]):
+// what a looped block adds ahead of a pass
+struct HyBranch { const float* y; const float* w; float mult; const int32_t* dst_of; int top; const float* add_rows = nullptr; const float* add_vec = nullptr; };
 cudaError_t hy_branch_norm(bool f32, float* x, const HyBranch& b, const int32_t* rows, const float* w, float eps, void* h, int ldh, int T, int W, cudaStream_t s);
 // x[t, c] *= sigmoid(g[t, c]) for c < n, in place (activation type)
 cudaError_t hy_sigmoid_gate(bool f32, void* x, int ldx, const void* g, int ldg, int n, int T, cudaStream_t s);
@@ -272,6 +280,8 @@ cudaError_t hy_sigmoid_gate(bool f32, void* x, int ldx, const void* g, int ldg, 
 cudaError_t hy_gather_rows_f32(const float* x, const int32_t* rows, float* out, int n, int W, cudaStream_t s);
 // softcap > 0: logits <- softcap * tanh(logits / softcap), in place, before the arg-max (ties -> lowest id)
 cudaError_t hy_argmax_rows(float* logits, int n, int V, float softcap, int32_t* out_ids, cudaStream_t s);
+// gu [T, ld]: gate and up products in alternating blocks of 16 columns -> out[t, f] = gelu_tanh(gate f) * (up f), f < ff
+cudaError_t hy_gelu_glu(bool f32, const void* gu, int ld, void* out, int ldo, int ff, int T, cudaStream_t s);
 // x[t, :] += v[:]
 cudaError_t hy_add_rowvec(float* x, const float* v, int T, int W, cudaStream_t s);
 

@@ -185,9 +185,10 @@ HybridModel::HybridModel(const ModelConfig& c, const EngineOptions& o) : ModelBa
     embed_ = upload_act(tensor("embed", V, W).v);
     head_ = upload_mat(tensor("head", V, W));
     final_norm_ = norm_weight("final.norm");
+    if (hc_.loop_times > 0 && hc_.loop_add) loop_step_ = upload_f32(vec("loop.step", hc_.loop_times * W, 0.f, 0.1f));
     if (hc_.loop_times > 0 && hc_.loop_reinject) { loop_in_ = upload_mat(tensor("loop.in", W, 2 * W)); loop_step_ = upload_f32(vec("loop.step", hc_.loop_times * W, 0.f, 0.1f)); }
     lw_.resize(hc_.layers.size());
-    int max_in = 8, max_p2 = 8, max_conv = 8, max_mix = 8, max_qabs = 8, max_lat = 8, max_qk = 8, max_v = 8, max_dec = 8, max_h = 8, max_act = 8, max_top = 1, max_E = 1, max_ffp = 16, max_lat_heads = 1, max_kv = 0, max_Eattn = 8, max_mix2 = 0, max_gates = 0, max_cq = 0;
+    int max_in = 8, max_p2 = 8, max_conv = 8, max_mix = 8, max_qabs = 8, max_lat = 8, max_qk = 8, max_v = 8, max_dec = 8, max_h = 8, max_act = 8, max_top = 1, max_E = 1, max_ffp = 16, max_lat_heads = 1, max_kv = 0, max_Eattn = 8, max_mix2 = 0, max_gates = 0, max_cq = 0, max_glu = 0;
     for (size_t li = 0; li < hc_.layers.size(); ++li) {
         const HyLayer& l = hc_.layers[li]; LayerW& w = lw_[li];
         const std::string p = "l" + std::to_string(li) + ".", mx = p + "mix.";
@@ -257,7 +258,7 @@ HybridModel::HybridModel(const ModelConfig& c, const EngineOptions& o) : ModelBa
                 while (rows % 8) { in.v.resize(in.v.size() + W, 0.f); ++rows; }
                 const int off = rows;
                 append_rows(in.v, rows, W, tensor(nm, nrows, W).v, nrows, 1);
-                if (two) { bias.resize(off, 0.f); std::vector<float> b = biased ? vec(nm + ".b", nrows, 0.f, 0.2f) : std::vector<float>(nrows, 0.f); bias.insert(bias.end(), b.begin(), b.end()); }
+                if (two && !l.scaled_sum) { bias.resize(off, 0.f); std::vector<float> b = biased ? vec(nm + ".b", nrows, 0.f, 0.2f) : std::vector<float>(nrows, 0.f); bias.insert(bias.end(), b.begin(), b.end()); }
                 return off;
             };
             if (two) {
@@ -265,9 +266,13 @@ HybridModel::HybridModel(const ModelConfig& c, const EngineOptions& o) : ModelBa
                     throw std::runtime_error("config.json: attention sizes beyond what the kernels hold (vdim <= 256)");
                 w.off_lq = seg(mx + "left.q", l.heads * l.dim, true); w.off_lk = seg(mx + "left.k", l.kv_heads * l.dim, true); w.off_lv = seg(mx + "left.v", l.kv_heads * l.vdim, true);
                 w.q_norm = upload_f32(vec(mx + "left.q.norm", l.heads * l.dim, 1.f, 0.1f)); w.k_norm = upload_f32(vec(mx + "left.k.norm", l.kv_heads * l.dim, 1.f, 0.1f));
-                w.o2 = upload_mat(tensor(mx + "left.o", W, l.heads * l.vdim)); w.o2_bias = upload_f32(vec(mx + "left.o.b", W, 0.f, 0.1f));
-                w.out_w1 = upload_f32(vec(mx + "left.out", W, 1.f, 0.1f)); w.out_w2 = upload_f32(vec(mx + "right.out", W, 1.f, 0.1f));
-                max_mix2 = std::max(max_mix2, l.heads * l.vdim);
+                if (l.scaled_sum) {
+                    if (l.rot_dims > 0) w.rope = rope_table(l.rot_base, l.rot_dims, l.rot_scaling.on ? &l.rot_scaling : nullptr);
+                } else {
+                    w.o2 = upload_mat(tensor(mx + "left.o", W, l.heads * l.vdim)); w.o2_bias = upload_f32(vec(mx + "left.o.b", W, 0.f, 0.1f));
+                    w.out_w1 = upload_f32(vec(mx + "left.out", W, 1.f, 0.1f)); w.out_w2 = upload_f32(vec(mx + "right.out", W, 1.f, 0.1f));
+                    max_mix2 = std::max(max_mix2, l.heads * l.vdim);
+                }
             }
             w.off_q = seg(lx + "q", qk, false);
             if (n.kind == HY_LIN_FORGET_WRITE) {        // [q | f | v]: the forget gate stands where the others keep their keys; no output gate
@@ -294,9 +299,23 @@ HybridModel::HybridModel(const ModelConfig& c, const EngineOptions& o) : ModelBa
                 w.gates_bias = upload_f32(gb); max_gates = std::max(max_gates, gr);
             }
             if (n.norm == HY_LIN_NORM_HEAD_WEIGHT) w.norm_w = upload_f32(vec(lx + "norm", n.vdim, 1.f, 0.1f));
-            else if (n.norm == HY_LIN_NORM_ALL_WEIGHT) w.norm_w = upload_f32(vec(lx + "norm", vd, 1.f, 0.1f));
-            if (two) { bias.resize(up8(rows), 0.f); w.in_bias = upload_f32(bias); w.in_bias_act = upload_act(bias); }
-            w.o = upload_mat(tensor(lx + "o", W, vd));
+            else if (n.norm == HY_LIN_NORM_ALL_WEIGHT || n.norm == HY_LIN_NORM_JOINT) {
+                std::vector<float> nw = vec(lx + "norm", vd, 1.f, 0.1f);
+                // a sum of two scaled outputs is one product over [left heads | right heads]: the left factor is the product's own, the right one relative to it rides in this norm's weight
+                if (l.scaled_sum) for (float& x : nw) x *= l.left_scale != 0.f ? l.right_scale / l.left_scale : l.right_scale;
+                w.norm_w = upload_f32(nw);
+            }
+            if (two && !l.scaled_sum) { bias.resize(up8(rows), 0.f); w.in_bias = upload_f32(bias); w.in_bias_act = upload_act(bias); }
+            if (l.scaled_sum) {        // [W_left | W_right] side by side, the right block on a multiple of 8 columns
+                const HostMat a = tensor(mx + "left.o", W, l.heads * l.vdim), b = tensor(lx + "o", W, vd);
+                w.off_mix2 = up8(a.K); w.o_alpha = l.left_scale != 0.f ? l.left_scale : 1.f;
+                HostMat o; o.N = W; o.K = w.off_mix2 + vd; o.v.assign((size_t)W * o.K, 0.f);
+                for (int i = 0; i < W; ++i) {
+                    if (l.left_scale != 0.f) std::memcpy(&o.v[(size_t)i * o.K], &a.v[(size_t)i * a.K], (size_t)a.K * 4);
+                    std::memcpy(&o.v[(size_t)i * o.K + w.off_mix2], &b.v[(size_t)i * vd], (size_t)vd * 4);
+                }
+                w.o = upload_mat(o); max_mix = std::max(max_mix, o.K);
+            } else w.o = upload_mat(tensor(lx + "o", W, vd));
             max_mix = std::max(max_mix, vd); max_qk = std::max(max_qk, qk); max_v = std::max(max_v, vd);
             max_dec = std::max(max_dec, n.kind == HY_LIN_CHANNEL_DECAY || n.kind == HY_LIN_FORGET_WRITE ? qk : n.heads); max_h = std::max(max_h, n.heads);
         } else if (l.type == HY_LATENT_ATTENTION) {
@@ -311,6 +330,10 @@ HybridModel::HybridModel(const ModelConfig& c, const EngineOptions& o) : ModelBa
             if (l.gate == HY_GATE_CHANNEL) {
                 while (rows % 8) { in.v.resize(in.v.size() + W, 0.f); ++rows; }
                 w.off_d = rows; append_rows(in.v, rows, W, tensor(mx + "g", l.heads * l.vdim, W).v, l.heads * l.vdim, 1);
+            }
+            if (l.gate == HY_GATE_HEAD) {
+                while (rows % 8) { in.v.resize(in.v.size() + W, 0.f); ++rows; }
+                w.off_d = rows; append_rows(in.v, rows, W, tensor(mx + "g", l.heads, W).v, l.heads, 1);
             }
             if (l.sink) w.sink = upload_f32(vec(mx + "sink", l.heads, 0.f, 1.f));
             w.dkv_norm = upload_f32(vec(mx + "dkv.norm", l.kv_rank, 1.f, 0.1f));
@@ -350,19 +373,27 @@ HybridModel::HybridModel(const ModelConfig& c, const EngineOptions& o) : ModelBa
             while (rows % 8) { in.v.resize(in.v.size() + W, 0.f); ++rows; }
             w.off_b = rows; append_rows(in.v, rows, W, tensor(mx + "b", l.heads, W).v, l.heads, 1);
             while (rows % 8) { in.v.resize(in.v.size() + W, 0.f); ++rows; }
-            HostMat a1 = tensor(mx + "a1", st_ ? (int)st_->st.get(mx + "a1").shape[0] : std::max(8, W / 16), W);
-            w.off_c = rows; w.a_rank = a1.N; append_rows(in.v, rows, W, a1.v, a1.N, 1);
-            while (rows % 8) { in.v.resize(in.v.size() + W, 0.f); ++rows; }
-            HostMat g1 = tensor(mx + "g1", st_ ? (int)st_->st.get(mx + "g1").shape[0] : std::max(8, W / 16), W);
-            w.off_d = rows; w.g_rank = g1.N; append_rows(in.v, rows, W, g1.v, g1.N, 1);
-            w.a2 = upload_mat(tensor(mx + "a2", l.heads * l.dim, w.a_rank)); w.g2 = upload_mat(tensor(mx + "g2", vd, w.g_rank));
-            w.A_log = upload_f32(vec(mx + "A_log", l.heads, 0.f, 0.5f)); w.dt_bias = upload_f32(vec(mx + "dt_bias", l.heads * l.dim, 0.f, 0.5f));
+            if (l.head_decay) {        // one decay per head and a full-rank gate: [a] and [g] are rows of the fused projection
+                w.off_c = rows; append_rows(in.v, rows, W, tensor(mx + "a", l.heads, W).v, l.heads, 1);
+                while (rows % 8) { in.v.resize(in.v.size() + W, 0.f); ++rows; }
+                w.off_d = rows; append_rows(in.v, rows, W, tensor(mx + "g", vd, W).v, vd, 1);
+                w.A_log = upload_f32(vec(mx + "A_log", l.heads, 0.f, 0.5f)); w.dt_bias = upload_f32(vec(mx + "dt_bias", l.heads, -2.f, 0.5f));
+            } else {
+                HostMat a1 = tensor(mx + "a1", st_ ? (int)st_->st.get(mx + "a1").shape[0] : std::max(8, W / 16), W);
+                w.off_c = rows; w.a_rank = a1.N; append_rows(in.v, rows, W, a1.v, a1.N, 1);
+                while (rows % 8) { in.v.resize(in.v.size() + W, 0.f); ++rows; }
+                HostMat g1 = tensor(mx + "g1", st_ ? (int)st_->st.get(mx + "g1").shape[0] : std::max(8, W / 16), W);
+                w.off_d = rows; w.g_rank = g1.N; append_rows(in.v, rows, W, g1.v, g1.N, 1);
+                w.a2 = upload_mat(tensor(mx + "a2", l.heads * l.dim, w.a_rank)); w.g2 = upload_mat(tensor(mx + "g2", vd, w.g_rank));
+                w.A_log = upload_f32(vec(mx + "A_log", l.heads, 0.f, 0.5f)); w.dt_bias = upload_f32(vec(mx + "dt_bias", l.heads * l.dim, 0.f, 0.5f));
+            }
             w.norm_w = upload_f32(vec(mx + "norm", l.vdim, 1.f, 0.1f));
             std::vector<float> cw = vec(mx + "q.conv", qk * l.conv, 0.f, 0.5f), ck = vec(mx + "k.conv", qk * l.conv, 0.f, 0.5f), cv = vec(mx + "v.conv", vd * l.conv, 0.f, 0.5f);
             cw.insert(cw.end(), ck.begin(), ck.end()); cw.insert(cw.end(), cv.begin(), cv.end());
             w.conv_w = upload_f32(cw);
             w.o = upload_mat(tensor(mx + "o", W, vd));
-            max_p2 = std::max(max_p2, up8(l.heads * l.dim) + vd); max_conv = std::max(max_conv, w.conv_ch); max_mix = std::max(max_mix, vd);
+            if (!l.head_decay) max_p2 = std::max(max_p2, up8(l.heads * l.dim) + vd);
+            max_conv = std::max(max_conv, w.conv_ch); max_mix = std::max(max_mix, vd);
             max_qk = std::max(max_qk, qk); max_v = std::max(max_v, vd); max_dec = std::max(max_dec, l.heads * l.dim); max_h = std::max(max_h, l.heads);
         } else {
             const int inner = l.heads * l.vdim, gn = l.groups * l.state, n_in = 2 * inner + 2 * gn + l.heads;
@@ -379,7 +410,17 @@ HybridModel::HybridModel(const ModelConfig& c, const EngineOptions& o) : ModelBa
         max_in = std::max(max_in, up8(rows));
         if (l.moe.present && l.moe.dense) {
             const std::string mp = p + "mlp.";
-            w.up = upload_mat(tensor(mp + "up", l.moe.ff, W)); w.dn = upload_mat(tensor(mp + "down", W, l.moe.ff));
+            if (l.moe.act == HY_EXPERT_GELU_GLU) {        // gate and up rows in alternating blocks of 16: the activation rides in the product's epilogue
+                const HostMat g = tensor(mp + "gate", l.moe.ff, W), u = tensor(mp + "up", l.moe.ff, W);
+                HostMat gu; w.ffp = up16(l.moe.ff); gu.N = 2 * w.ffp; gu.K = W; gu.v.assign((size_t)gu.N * W, 0.f);
+                for (int f = 0; f < l.moe.ff; ++f) {
+                    const size_t at = (size_t)((f >> 4) * 32 + (f & 15)) * W;
+                    std::memcpy(&gu.v[at], &g.v[(size_t)f * W], (size_t)W * 4); std::memcpy(&gu.v[at + (size_t)16 * W], &u.v[(size_t)f * W], (size_t)W * 4);
+                }
+                w.up = upload_mat(gu); max_act = std::max(max_act, w.ffp);
+                if (!w.up.tc) max_glu = std::max(max_glu, gu.N);
+            } else w.up = upload_mat(tensor(mp + "up", l.moe.ff, W));
+            w.dn = upload_mat(tensor(mp + "down", W, l.moe.ff));
             if (l.moe.act == HY_EXPERT_POLY_NORM) { const std::vector<float> a = vec(mp + "act", 4, 0.5f, 0.4f); w.poly = HyPolyCoef{a[0], a[1], a[2], a[3]}; }
             max_act = std::max(max_act, up8(l.moe.ff));
         } else if (l.moe.present) {
@@ -463,6 +504,7 @@ HybridModel::HybridModel(const ModelConfig& c, const EngineOptions& o) : ModelBa
         tile_expert_ = (int32_t*)dmalloc((size_t)max_tiles_ * 4); row_src_ = (int32_t*)dmalloc((size_t)max_tiles_ * 128 * 4);
         n_tiles_ = (int32_t*)dmalloc((size_t)(4 + 2 * max_E) * 4); dst_of_ = (int32_t*)dmalloc(MR * max_top * 4);
     }
+    if (max_glu > 0) { ld_glu_ = max_glu; glu_ = dmalloc(MR * ld_glu_ * es_); }
     if (hc_.post_norm) { y_ = (float*)dmalloc(MR * W * 4); y2_ = (float*)dmalloc(MR * W * 4); }
     if (hc_.sequential) {
         n_streams_ = std::max(1, hc_.streams);
@@ -547,18 +589,18 @@ static int pick_tile_n(int M, int N, int sms) {
 }
 static bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 
-void HybridModel::gemm(int mode, const void* A, int lda, const Mat& B, void* C, int ldc, int M, const float* bias, float alpha, const void* bias_act, int act) {
+void HybridModel::gemm(int mode, const void* A, int lda, const Mat& B, void* C, int ldc, int M, const float* bias, float alpha, const void* bias_act, HyGemmAct act) {
     // bf16: the framework's tcgen05 tile GEMM (TMA operands, fp32 accumulator in TMEM) wherever pitches and pointers fit its 16-byte rules;
     // a bf16 store may write the columns up to N rounded up to 8 (every such output has that room), an fp32 output needs N itself to fit
     bool tc = B.tc && !f32_ && lda % 8 == 0 && aligned16(A) && lda >= B.ld;
     if (mode == HY_STORE) tc = tc && ldc % 8 == 0 && aligned16(C) && (!bias || (bias_act && aligned16(bias_act))) && alpha == 1.f;     // a bias in the activation type, padded to N rounded up to 8
-    else tc = tc && B.N % 8 == 0 && ldc % 4 == 0 && aligned16(C) && (!bias || aligned16(bias)) && act == 0;
+    else tc = tc && B.N % 8 == 0 && ldc % 4 == 0 && aligned16(C) && (!bias || aligned16(bias)) && act.kind == 0;
     CUtensorMap tmA;
     if (tc && make_tmap_bf16_2d(&tmA, A, (uint64_t)M, (uint64_t)B.ld, (uint64_t)lda, 128, 64) != 0) tc = false;
     if (!tc) { cuda_check(hy_gemm(f32_, mode, A, lda, B.p, B.ld, C, ldc, M, B.N, B.K, bias, alpha, 1, 0, 0, 0, stream, act), "gemm"); return; }
     GemmParams g{}; g.M = M; g.N = up8(B.N); g.K = B.ld;
     const int bn = pick_tile_n(M, g.N, sm_count);
-    if (mode == HY_STORE) { g.out = C; g.ldo = ldc; g.bias = bias ? bias_act : nullptr; g.store_act = act; cuda_check(launch_gemm(&tmA, &B.tm[bn == 32 ? 0 : bn == 64 ? 1 : bn == 128 ? 2 : 3], g, EPI_STORE, bn, stream), "gemm (tcgen05)"); return; }
+    if (mode == HY_STORE) { g.out = C; g.ldo = ldc; g.bias = bias ? bias_act : nullptr; g.store_act = act.kind; g.act_col0 = act.col0; g.act_col1 = act.col1; cuda_check(launch_gemm(&tmA, &B.tm[bn == 32 ? 0 : bn == 64 ? 1 : bn == 128 ? 2 : 3], g, EPI_STORE, bn, stream), "gemm (tcgen05)"); return; }
     g.f32_out = reinterpret_cast<float*>(C); g.ldf = ldc; g.f32_accumulate = mode == HY_ACC_F32; g.alpha = alpha; g.bias_f32 = bias;
     cuda_check(launch_gemm(&tmA, &B.tm[bn == 32 ? 0 : bn == 64 ? 1 : bn == 128 ? 2 : 3], g, EPI_F32, bn, stream), "gemm (tcgen05, fp32 out)");
 }
@@ -568,8 +610,23 @@ bool HybridModel::moe(const LayerW& w, const HyLayer& l, const void* h_in, const
     float* out = x_;
     if (hc_.sequential) { out = y_; beta = 0.f; }        // the residual is closed by whoever opens the next sublayer
     const bool relu2 = m.act == HY_EXPERT_RELU2; const int rows1 = relu2 ? w.ffp : 2 * w.ffp;
+    if (m.dense && m.act == HY_EXPERT_GELU_GLU) {        // gated: both halves in one product, gelu(gate) * up in its epilogue
+        CUtensorMap tmA;
+        if (w.up.tc && make_tmap_bf16_2d(&tmA, h_in, (uint64_t)T, (uint64_t)w.up.ld, (uint64_t)Wld_, 128, 64) == 0) {
+            GemmParams g{}; g.M = T; g.N = w.up.N; g.K = w.up.ld; g.out = act_; g.ldo = w.ffp; g.glu_gelu = 1;
+            const int bn = pick_tile_n(T, g.N, sm_count);
+            cuda_check(launch_gemm(&tmA, &w.up.tm[bn == 32 ? 0 : bn == 64 ? 1 : bn == 128 ? 2 : 3], g, EPI_SWIGLU, bn, stream), "gated feed-forward (tcgen05)");
+        } else {
+            if (!glu_) throw std::runtime_error("tensor map for the feed-forward's input failed");
+            gemm(HY_STORE, h_in, Wld_, w.up, glu_, ld_glu_, T, nullptr, 1.f);
+            cuda_check(hy_gelu_glu(f32_, glu_, ld_glu_, act_, w.ffp, w.ffp, T, stream), "gated activation");
+        }
+        MARK(25);
+        gemm(HY_STORE_F32, act_, w.ffp, w.dn, y_, W, T, nullptr, 1.f); MARK(26);
+        return false;
+    }
     if (m.dense) {        // one feed-forward for every row: up product with the activation in its epilogue, down product into the sublayer's fp32 output
-        gemm(HY_STORE, h_in, Wld_, w.up, act_, up8(m.ff), T, nullptr, 1.f, nullptr, relu2 ? 1 : m.act == HY_EXPERT_GELU_TANH ? 2 : 0); MARK(25);
+        gemm(HY_STORE, h_in, Wld_, w.up, act_, up8(m.ff), T, nullptr, 1.f, nullptr, HyGemmAct{relu2 ? 1 : m.act == HY_EXPERT_GELU_TANH ? 2 : 0}); MARK(25);
         if (m.act == HY_EXPERT_POLY_NORM) { cuda_check(hy_poly_norm(f32_, act_, up8(m.ff), m.ff, w.poly, hc_.eps, T, stream), "poly norm"); MARK(30); }
         gemm(HY_STORE_F32, act_, up8(m.ff), w.dn, y_, W, T, nullptr, 1.f); MARK(26);
         return false;
@@ -652,6 +709,10 @@ void HybridModel::linear_mixer(const HyRun& run, const HyLayer& l, const LayerW&
         const float* rc = w.rope >= 0 ? ropes_[w.rope].cos : nullptr; const float* rs = w.rope >= 0 ? ropes_[w.rope].sin : nullptr;
         cuda_check(hy_lin_prep(f32_, HyLinPrep{H, D, VD, n.q_scaled, n.k_scaled, n.rot_dims}, q, k, v, ld_proj_, qq_, kk_, vv_, nullptr, 1.f, w.decay, dec_, rc, rs, r, stream), "retention operands"); MARK(28);
         cuda_check(hy_recurrence(HY_REC_SCALAR, qq_, kk_, vv_, dec_, nullptr, rec_, st, H, H, D, VD, r, stream), "retention"); MARK(8);
+        if (n.norm == HY_LIN_NORM_JOINT) {       // one norm over all heads; a layer that joins two mixers puts it behind the attention side's heads
+            cuda_check(hy_gated_norm(f32_, rec_, H * VD, H * VD, w.norm_w, H * VD, g, ld_proj_, 0, n.gate_silu, nullptr, 1, nullptr, 0, at(mix_, w.off_mix2), ld_mix_, hc_.eps, T, stream), "joint norm"); MARK(9);
+            return;
+        }
         cuda_check(hy_gated_norm(f32_, rec_, H * VD, VD, nullptr, 1, g, ld_proj_, 0, n.gate_silu, nullptr, 1, nullptr, 0, mix_, ld_mix_, hc_.eps, T, stream), "gated norm"); MARK(9);
     } else {
         float* aux = aux_[run.state_idx];
@@ -663,6 +724,35 @@ void HybridModel::linear_mixer(const HyRun& run, const HyLayer& l, const LayerW&
     }
 }
 
+
+// attention side of a layer with two mixers, cache row written: queries q [T, ld] -> heads' outputs in out
+void HybridModel::attend(const HyWinAttn& a, void* q, int ld, const HyRun& run, const HyRows& r, const TileList& tl, void* out, int ldo) {
+    void* cache = caches_[run.cache_idx];
+    if (tl.mma) {
+        cuda_check(hy_win_attention_mma(a, q, ld, cache, nullptr, nullptr, 0, out, ldo, hc_.eps, r, d_meta_ + tl.o_wseq, d_meta_ + tl.o_wq0, tl.n_w, stream), "attention (mma)");
+        cuda_check(hy_win_decode_mma(a, q, ld, cache, nullptr, nullptr, 0, out, ldo, hc_.eps, r, d_meta_ + tl.o_dseq, d_meta_ + tl.o_dq0, tl.n_d, stream), "attention (mma, decoding rows)");
+    } else cuda_check(hy_win_attention(f32_, a, q, ld, cache, nullptr, nullptr, 0, out, ldo, hc_.eps, r, stream), "attention");
+}
+
+// Gated delta rule: short convolutions, operands, the recurrence on the sequence's state slot, the norm per head with its output gate; leaves the
+// output projection's input in mix_.  A decay per key channel comes with low-rank second stages for decay and gate, one decay per head with neither.
+void HybridModel::delta_mixer(const HyRun& run, const HyLayer& l, const LayerW& w, const HyRows& r, const std::function<void(int)>& MARK) {
+    const int T = r.T;
+    auto at = [&](void* base, size_t elems) -> void* { return reinterpret_cast<char*>(base) + elems * es_; };
+    const HyDelta d{l.heads, l.kv_heads, l.dim, l.vdim, l.head_decay};
+    cuda_check(hy_conv_silu(f32_, at(proj_, w.off_a), ld_proj_, w.conv_ch, w.conv_w, nullptr, l.conv, conv_, ld_conv_, tails_[run.state_idx], r, stream), "conv");
+    cuda_check(hy_conv_tails(f32_, at(proj_, w.off_a), ld_proj_, w.conv_ch, l.conv, tails_[run.state_idx], r, stream), "conv tails"); MARK(6);
+    const void *a = at(proj_, w.off_c), *g = at(proj_, w.off_d); int ld_a = ld_proj_, ld_g = ld_proj_;
+    if (!l.head_decay) {
+        const int off_g = up8(l.heads * l.dim);
+        gemm(HY_STORE, at(proj_, w.off_c), ld_proj_, w.a2, p2_, ld_p2_, T, nullptr, 1.f);
+        gemm(HY_STORE, at(proj_, w.off_d), ld_proj_, w.g2, at(p2_, off_g), ld_p2_, T, nullptr, 1.f); MARK(10);
+        a = p2_; g = at(p2_, off_g); ld_a = ld_g = ld_p2_;
+    }
+    cuda_check(hy_delta_prep(f32_, d, conv_, ld_conv_, at(proj_, w.off_b), ld_proj_, a, ld_a, w.A_log, w.dt_bias, qq_, kk_, vv_, dec_, beta_, T, stream), "delta prep"); MARK(7);
+    cuda_check(hy_recurrence(l.head_decay ? HY_REC_DELTA_HEAD : HY_REC_DELTA, qq_, kk_, vv_, dec_, beta_, rec_, states_[run.state_idx], l.heads, l.kv_heads, l.dim, l.vdim, r, stream), "delta rule"); MARK(8);
+    cuda_check(hy_gated_norm(f32_, rec_, l.heads * l.vdim, l.vdim, w.norm_w, l.vdim, g, ld_g, 0, l.head_decay, nullptr, 1, nullptr, 0, mix_, ld_mix_, hc_.eps, T, stream), "gated norm"); MARK(9);
+}
 
 HyLatentAttn HybridModel::latent_params(const HyLayer& l, const LayerW& w) const {
     HyLatentAttn a{l.heads, l.dim, l.rot_dim, l.vdim, l.kv_rank, l.rot_dims, l.scale};
@@ -698,7 +788,8 @@ void HybridModel::latent_mixer(const HyRun& run, const HyLayer& l, const LayerW&
                                const void* gate, int ldg) {
     auto at = [&](void* base, size_t elems) -> void* { return reinterpret_cast<char*>(base) + elems * es_; };
     const int T = r.T;
-    const HyLatentAttn a = latent_params(l, w);
+    HyLatentAttn a = latent_params(l, w);
+    if (l.gate == HY_GATE_HEAD) { a.head_gate = gate; a.ldg = ldg; gate = nullptr; }        // a factor per head rides in the attention kernels' epilogues
     const int E = l.kv_rank + l.rot_dim;
     cuda_check(hy_mla_prep(f32_, a, q, ldq, ckv, ldc, w.dkv_norm, hc_.eps, ropes_[w.rope].cos, ropes_[w.rope].sin, caches_[run.cache_idx], q_abs_, r, stream), "latent cache write"); MARK(4);
     if (tl.any_small) {
@@ -712,7 +803,7 @@ void HybridModel::latent_mixer(const HyRun& run, const HyLayer& l, const LayerW&
             HyMlaSplit sp{nullptr, nullptr, nullptr, split_o_, split_ml_};
             if (tl.n_merge > 0) { sp.tile_k0 = d_meta_ + tl.o_k0; sp.tile_k1 = d_meta_ + tl.o_k1; sp.tile_slot = d_meta_ + tl.o_slot; }
             cuda_check(hy_mla_attention_mma(a, q_abs_, caches_[run.cache_idx], lat_, r, d_meta_ + tl.o_seq, d_meta_ + tl.o_q0, tl.n, sp, stream), "latent attention (mma)");
-            cuda_check(hy_mla_merge(d_meta_ + tl.o_mrow, d_meta_ + tl.o_mslot, d_meta_ + tl.o_mparts, tl.n_merge, split_o_, split_ml_, lat_, l.heads, l.kv_rank, stream, a.sink), "latent attention (join)");
+            cuda_check(hy_mla_merge(d_meta_ + tl.o_mrow, d_meta_ + tl.o_mslot, d_meta_ + tl.o_mparts, tl.n_merge, split_o_, split_ml_, lat_, l.heads, l.kv_rank, stream, a.sink, a.head_gate, a.ldg), "latent attention (join)");
         } else cuda_check(hy_mla_attention(f32_, a, q_abs_, caches_[run.cache_idx], lat_, r, stream), "latent attention");
         MARK(5);
         if (head_tc) for (int hd = 0; hd < l.heads; ++hd) gemm(HY_STORE, at(lat_, (size_t)hd * l.kv_rank), l.heads * l.kv_rank, w.uv_heads[hd], at(mix_, (size_t)hd * l.vdim), ld_mix_, T, nullptr, 1.f);
@@ -741,10 +832,11 @@ void HybridModel::forward_sequential(const HyRows& r, const std::vector<TileList
     const float *pend_mix = nullptr, *pend_out = nullptr;      // coefficients of the sublayer whose y_ has not been folded into the streams yet
     bool pending = false;
     HyBranch branch{nullptr, nullptr, hc_.residual_mult, nullptr, 0};        // designs with a norm behind the sublayer: the one that has not joined the residual yet
+    if (hc_.single_stream) branch.mult = 1.f;
     auto open = [&](const float* in, const float* norm_w, float* shift_state, const char* what) {
-        if (hc_.branch_norm) {
+        if (hc_.branch_norm || hc_.single_stream) {
             cuda_check(hy_branch_norm(f32_, xs_, branch, nullptr, norm_w, hc_.eps, h_, Wld_, T, W, stream), what);
-            branch.y = nullptr;
+            branch.y = branch.add_rows = branch.add_vec = nullptr;
             return;
         }
         const HyStreams c{n, pend_mix, pend_out, in};
@@ -754,10 +846,12 @@ void HybridModel::forward_sequential(const HyRows& r, const std::vector<TileList
     for (const HyRun& run : hc_.runs) {
         const HyLayer& l = hc_.layers[run.layer]; const LayerW& w = lw_[run.layer];
         float* sstate = w.shift ? shift_states_[run.index] : nullptr;
+        if (hc_.loop_add && run.first_of_pass) { branch.add_rows = run.pass > 0 ? x0_ : nullptr; branch.add_vec = loop_step_ + (size_t)run.pass * W; }      // joins the residual with the sublayer that is closed here
         open(hyper ? w.hc_in[0] : ones_, w.norm1, sstate, "streams + norm (mixer)");
         if (sstate) cuda_check(hy_token_shift(f32_, hn_, shift_prev_, w.shift, h_, Wld_, r, W, stream), "token shift");
         MARK(hc_.branch_norm ? 31 : 22);
-        gemm(HY_STORE, h_, Wld_, w.in, proj_, ld_proj_, T, w.in_bias, 1.f, w.in_bias_act); MARK(2);
+        const HyGemmAct in_act = l.lin.qkv_silu ? HyGemmAct{3, w.off_q, w.off_g} : HyGemmAct();       // lightning attention's q | k | v, padding columns included
+        gemm(HY_STORE, h_, Wld_, w.in, proj_, ld_proj_, T, w.in_bias, 1.f, w.in_bias_act, in_act); MARK(2);
         if (l.type == HY_LINEAR_ATTENTION) linear_mixer(run, l, w, r, MARK);
         else if (l.type == HY_LATENT_ATTENTION) {
             void* q = at(proj_, w.off_a); int ldq = ld_proj_;
@@ -766,7 +860,16 @@ void HybridModel::forward_sequential(const HyRows& r, const std::vector<TileList
                 gemm(HY_STORE, cq_, ld_cq_, w.uq, p2_, ld_p2_, T, nullptr, 1.f); MARK(10);
                 q = p2_; ldq = ld_p2_;
             }
-            latent_mixer(run, l, w, r, tile_lists[run.layer], MARK, q, ldq, at(proj_, w.off_b), ld_proj_, l.gate == HY_GATE_CHANNEL ? at(proj_, w.off_d) : nullptr, ld_proj_);
+            latent_mixer(run, l, w, r, tile_lists[run.layer], MARK, q, ldq, at(proj_, w.off_b), ld_proj_, l.gate ? at(proj_, w.off_d) : nullptr, ld_proj_);
+        } else if (l.type == HY_CHANNEL_DELTA) delta_mixer(run, l, w, r, MARK);
+        else if (l.type == HY_ATTENTION_BESIDE_MEMORY) {
+            const HyWinAttn a = window_params(l, w); const TileList& tl = tile_lists[run.layer];
+            const HyRotary rot{l.rot_dims, l.rot_layout, l.rot_dims > 0 ? ropes_[w.rope].cos : nullptr, l.rot_dims > 0 ? ropes_[w.rope].sin : nullptr, nullptr, nullptr};
+            void* q = at(proj_, w.off_lq);
+            cuda_check(hy_win_prep(f32_, a, q, ld_proj_, at(proj_, w.off_lk), at(proj_, w.off_lv), ld_proj_, w.q_norm, w.k_norm, hc_.eps, caches_[run.cache_idx], r, stream, &rot),
+                       "query / key norm + rotary + cache write"); MARK(23);
+            attend(a, q, ld_proj_, run, r, tl, mix_, ld_mix_); MARK(24);
+            linear_mixer(run, l, w, r, MARK);
         } else if (l.type == HY_WINDOW_ATTENTION) {
             void* src = proj_; int ld = ld_proj_;
             const HyWinAttn wa = window_params(l, w);
@@ -787,7 +890,7 @@ void HybridModel::forward_sequential(const HyRows& r, const std::vector<TileList
             window_mixer(run, l, w, r, tile_lists[run.layer], MARK, at(src, w.off_a), at(src, w.off_b), at(src, w.off_c), ld, l.gate ? at(proj_, w.off_d) : nullptr, ld_proj_);
             }
         } else throw std::runtime_error("forward: this design has no such mixer");
-        gemm(HY_STORE_F32, mix_, ld_mix_, w.o, y_, W, T, w.o_bias, 1.f); MARK(11);
+        gemm(HY_STORE_F32, mix_, ld_mix_, w.o, y_, W, T, w.o_bias, w.o_alpha); MARK(11);
         pending = true; pend_mix = hyper ? w.hc_mix[0] : ones_; pend_out = hyper ? w.hc_out[0] : ones_;
         branch.y = y_; branch.w = w.norm1b; branch.dst_of = nullptr;
         if (l.moe.present) {
@@ -841,7 +944,7 @@ void HybridModel::forward(const StepInput& in, float* logits_out) {
         const HyLayer& l = hc_.layers[li]; TileList& tl = tile_lists[li];
         if (l.type == HY_WINDOW_ATTENTION || l.type == HY_ATTENTION_BESIDE_MEMORY) {
             // windowed attention on the tensor cores: tiles of 64 consecutive (row, head-of-the-group) pairs of one sequence; a decoding row is one tile per key/value head
-            tl.mma = !f32_ && opt.hy_tensor_core && ld_proj_ % 8 == 0 && (l.type == HY_WINDOW_ATTENTION ? ld_mix_ : ld_mix2_) % 8 == 0 && hy_win_mma_supported(window_params(l, lw_[li]));
+            tl.mma = !f32_ && opt.hy_tensor_core && ld_proj_ % 8 == 0 && (l.type == HY_WINDOW_ATTENTION || l.scaled_sum ? ld_mix_ : ld_mix2_) % 8 == 0 && hy_win_mma_supported(window_params(l, lw_[li]));
             if (!tl.mma) continue;
             tile_seq_.clear(); tile_q0_.clear(); ptile_seq_.clear(); ptile_row0_.clear();
             const int group = l.heads / l.kv_heads;
@@ -910,7 +1013,8 @@ void HybridModel::forward(const StepInput& in, float* logits_out) {
         cudaEventRecord(ev_all[ek++], stream);
     }
     const std::function<void(int)> MARK = [&](int id) { if (profile_all && ek < ev_all.size()) { ev_ids[ek] = id; cudaEventRecord(ev_all[ek++], stream); } };
-    if (hc_.sequential) { cuda_check(hy_embed_streams(f32_, d_meta_ + o_tok, embed_, xs_, T, W, V, hc_.embed_scale, n_streams_, stream), "embed"); MARK(0); forward_sequential(r, tile_lists, d_meta_ + o_tok, MARK); }
+    if (hc_.single_stream) { cuda_check(hy_embed(f32_, d_meta_ + o_tok, embed_, xs_, hc_.loop_times > 0 ? x0_ : nullptr, T, W, V, hc_.embed_scale, stream, nullptr, 0), "embed"); MARK(0); forward_sequential(r, tile_lists, d_meta_ + o_tok, MARK); }
+    else if (hc_.sequential) { cuda_check(hy_embed_streams(f32_, d_meta_ + o_tok, embed_, xs_, T, W, V, hc_.embed_scale, n_streams_, stream), "embed"); MARK(0); forward_sequential(r, tile_lists, d_meta_ + o_tok, MARK); }
     else { cuda_check(hy_embed(f32_, d_meta_ + o_tok, embed_, x_, hc_.loop_times > 0 ? x0_ : nullptr, T, W, V, hc_.embed_scale, stream, hc_.post_norm ? h_ : nullptr, Wld_), "embed"); MARK(0); }
     auto at = [&](void* base, size_t elems) -> void* { return reinterpret_cast<char*>(base) + elems * es_; };
     for (const HyRun& run : hc_.runs) {
@@ -929,14 +1033,7 @@ void HybridModel::forward(const StepInput& in, float* logits_out) {
                 const HyWinAttn a = window_params(l, w);
                 cuda_check(hy_win_prep(f32_, a, at(proj_, w.off_lq), ld_proj_, at(proj_, w.off_lk), at(proj_, w.off_lv), ld_proj_, w.q_norm, w.k_norm, hc_.eps, caches_[run.cache_idx], r, stream),
                            "query / key norm + cache write"); MARK(23);
-                const TileList& tl = tile_lists[run.layer];
-                if (tl.mma) {
-                    cuda_check(hy_win_attention_mma(a, at(proj_, w.off_lq), ld_proj_, caches_[run.cache_idx], nullptr, nullptr, 0, mix2_, ld_mix2_, hc_.eps, r, d_meta_ + tl.o_wseq, d_meta_ + tl.o_wq0,
-                                                    tl.n_w, stream), "attention (mma)");
-                    cuda_check(hy_win_decode_mma(a, at(proj_, w.off_lq), ld_proj_, caches_[run.cache_idx], nullptr, nullptr, 0, mix2_, ld_mix2_, hc_.eps, r, d_meta_ + tl.o_dseq, d_meta_ + tl.o_dq0,
-                                                 tl.n_d, stream), "attention (mma, decoding rows)");
-                } else cuda_check(hy_win_attention(f32_, a, at(proj_, w.off_lq), ld_proj_, caches_[run.cache_idx], nullptr, nullptr, 0, mix2_, ld_mix2_, hc_.eps, r, stream), "attention");
-                MARK(24);
+                attend(a, at(proj_, w.off_lq), ld_proj_, run, r, tile_lists[run.layer], mix2_, ld_mix2_); MARK(24);
                 gemm(HY_STORE_F32, mix2_, ld_mix2_, w.o2, y2_, W, T, w.o2_bias, 1.f); MARK(11);
             }
             linear_mixer(run, l, w, r, MARK);
@@ -967,15 +1064,7 @@ void HybridModel::forward(const StepInput& in, float* logits_out) {
         } else if (l.type == HY_LATENT_ATTENTION) {
             latent_mixer(run, l, w, r, tile_lists[run.layer], MARK, at(proj_, w.off_a), ld_proj_, at(proj_, w.off_b), ld_proj_);
         } else if (l.type == HY_CHANNEL_DELTA) {
-            const HyDelta d{l.heads, l.kv_heads, l.dim, l.vdim};
-            cuda_check(hy_conv_silu(f32_, at(proj_, w.off_a), ld_proj_, w.conv_ch, w.conv_w, nullptr, l.conv, conv_, ld_conv_, tails_[run.state_idx], r, stream), "conv");
-            cuda_check(hy_conv_tails(f32_, at(proj_, w.off_a), ld_proj_, w.conv_ch, l.conv, tails_[run.state_idx], r, stream), "conv tails"); MARK(6);
-            const int off_g = up8(l.heads * l.dim);
-            gemm(HY_STORE, at(proj_, w.off_c), ld_proj_, w.a2, p2_, ld_p2_, T, nullptr, 1.f);
-            gemm(HY_STORE, at(proj_, w.off_d), ld_proj_, w.g2, at(p2_, off_g), ld_p2_, T, nullptr, 1.f); MARK(10);
-            cuda_check(hy_delta_prep(f32_, d, conv_, ld_conv_, at(proj_, w.off_b), ld_proj_, p2_, ld_p2_, w.A_log, w.dt_bias, qq_, kk_, vv_, dec_, beta_, T, stream), "delta prep"); MARK(7);
-            cuda_check(hy_recurrence(HY_REC_DELTA, qq_, kk_, vv_, dec_, beta_, rec_, states_[run.state_idx], l.heads, l.kv_heads, l.dim, l.vdim, r, stream), "delta rule"); MARK(8);
-            cuda_check(hy_gated_norm(f32_, rec_, l.heads * l.vdim, l.vdim, w.norm_w, l.vdim, at(p2_, off_g), ld_p2_, 0, 0, nullptr, 1, nullptr, 0, mix_, ld_mix_, hc_.eps, T, stream), "gated norm"); MARK(9);
+            delta_mixer(run, l, w, r, MARK);
         } else {
             const HyMamba m{l.heads, l.vdim, l.state, l.groups};
             const int inner = l.heads * l.vdim;
@@ -999,7 +1088,7 @@ void HybridModel::forward(const StepInput& in, float* logits_out) {
         capture_layers = nullptr;
     }
     if (NS > 0) {
-        if (hc_.branch_norm) {
+        if (hc_.branch_norm || hc_.single_stream) {
             cuda_check(hy_branch_norm(f32_, xs_, pend_branch_, d_meta_ + o_samp, final_norm_, hc_.eps, hs_, Wld_, NS, W, stream), "final norm");
         } else if (hc_.sequential) {      // x = the sum of the streams, of the wanted rows only
             const HyStreams fin{n_streams_, pend_mix_, pend_out_, ones_};

@@ -58,6 +58,7 @@ private:
         // linear attention and attention beside a matrix memory: segments of the fused input projection, second stage and biases
         int off_q = 0, off_k = 0, off_v = 0, off_g = 0, off_a1 = 0, off_lq = 0, off_lk = 0, off_lv = 0;
         float *a2_bias = nullptr, *decay = nullptr, *o2_bias = nullptr, *out_w1 = nullptr, *out_w2 = nullptr, *gates_bias = nullptr;
+        int off_mix2 = 0; float o_alpha = 1.f;        // a sum of two scaled mixers as one product: column of the second one's heads, factor of the whole
         Mat o2, gates;                                // output projection of the attention side; [W_i ; W_f] of the matrix memory (fp32 out)
     };
     struct RopeTable { float base; int dims; HyRotScaling sc; float *cos = nullptr, *sin = nullptr; };
@@ -74,7 +75,7 @@ private:
     std::vector<float> vec(const std::string& name, int n, float init_mean, float init_spread);
     float* norm_weight(const std::string& name);                          // [width] weight of a layer norm or the final norm as it multiplies (stored around one or around zero)
     void distance_bias(LayerW& w, const HyLayer& l, const std::string& name);      // bias table [rows, heads] -> one entry per distance
-    void gemm(int mode, const void* A, int lda, const Mat& B, void* C, int ldc, int M, const float* bias, float alpha, const void* bias_act = nullptr, int act = 0);
+    void gemm(int mode, const void* A, int lda, const Mat& B, void* C, int ldc, int M, const float* bias, float alpha, const void* bias_act = nullptr, HyGemmAct act = HyGemmAct());
     // routed experts (and a dense feed-forward): x = beta x + sum of the chosen experts' outputs (sequential designs: the sum alone goes to y_).
     // Returns true where the caller is to add the choices itself: their rows lie in moe_y_ at dst_of_ (designs with a norm behind the sublayer)
     bool moe(const LayerW& w, const HyLayer& l, const void* h, const HyRows& r, const std::function<void(int)>& mark, const int32_t* tokens = nullptr, float beta = 1.f);
@@ -89,6 +90,8 @@ private:
     HyWinAttn window_params(const HyLayer& l, const LayerW& w) const;
     HyLatentAttn latent_params(const HyLayer& l, const LayerW& w) const;
     void linear_mixer(const HyRun& run, const HyLayer& l, const LayerW& w, const HyRows& r, const std::function<void(int)>& mark);
+    void delta_mixer(const HyRun& run, const HyLayer& l, const LayerW& w, const HyRows& r, const std::function<void(int)>& mark);
+    void attend(const HyWinAttn& a, void* q, int ld, const HyRun& run, const HyRows& r, const TileList& tl, void* out, int ldo);
     bool has_tensor(const std::string& name) const;
     int cache_row_width(const HyLayer& l) const { return (l.type == HY_WINDOW_ATTENTION || l.type == HY_ATTENTION_BESIDE_MEMORY) ? l.kv_heads * (l.maps * l.dim + l.vdim) : l.kv_rank + l.rot_dim; }
 
@@ -112,6 +115,7 @@ private:
     void *cat_ = nullptr, *h_ = nullptr, *h2_ = nullptr, *proj_ = nullptr, *p2_ = nullptr, *conv_ = nullptr, *lat_ = nullptr, *mix_ = nullptr, *act_ = nullptr, *hs_ = nullptr, *moe_a_ = nullptr;
     int ld_proj_ = 0, ld_p2_ = 0, ld_conv_ = 0, ld_mix_ = 0, ld_mix2_ = 0, ld_gates_ = 0;
     float *y_ = nullptr, *y2_ = nullptr, *gates_ = nullptr, *gin_ = nullptr, *floor_ = nullptr, *ndot_ = nullptr;     // post-norm designs: sublayer outputs; matrix memory: gates and normaliser terms
+    void* glu_ = nullptr; int ld_glu_ = 0;         // gate and up products of a gated dense feed-forward where the activation is a kernel of its own
     void* mix2_ = nullptr;                         // attention side of a layer with two mixers
     int32_t *idx_ = nullptr, *d_out_ids_ = nullptr, *tile_expert_ = nullptr, *row_src_ = nullptr, *n_tiles_ = nullptr, *dst_of_ = nullptr; int max_tiles_ = 0;
     int32_t* h_meta_buf_[2] = {nullptr, nullptr}; cudaEvent_t meta_ev_[2] = {nullptr, nullptr}; int meta_idx_ = 0;

@@ -192,6 +192,22 @@ __device__ __forceinline__ void branch_load(const HyBranch& b, long long src, in
         for (int e = 0; e < V; ++e) y.v[e] += u.v[e];
     }
 }
+// what a looped block adds to a row ahead of a pass
+template <int V>
+__device__ __forceinline__ FVec<V> branch_add(const HyBranch& b, long long src, int W, int c, FVec<V> v) {
+    FVec<V> u;
+    if (b.add_rows) {
+        u.load(b.add_rows + src * W + c);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v.v[e] += u.v[e];
+    }
+    if (b.add_vec) {
+        u.load(b.add_vec + c);
+#pragma unroll
+        for (int e = 0; e < V; ++e) v.v[e] += u.v[e];
+    }
+    return v;
+}
 template <typename TA, int NV>      // NV float4 per thread: W <= 1024 NV
 __global__ void __launch_bounds__(256) hy_branch_norm_reg_kernel(float* __restrict__ x, HyBranch b, const int32_t* __restrict__ rows, const float* __restrict__ w, float eps,
                                                                  TA* __restrict__ h, int ldh, int W) {
@@ -209,18 +225,27 @@ __global__ void __launch_bounds__(256) hy_branch_norm_reg_kernel(float* __restri
             const int c = (threadIdx.x + k * 256) * 4;
             if (c < W) { branch_load<4>(b, src, W, c, y[k]); ss += (y[k].v[0] * y[k].v[0] + y[k].v[1] * y[k].v[1]) + (y[k].v[2] * y[k].v[2] + y[k].v[3] * y[k].v[3]); }
         }
-        const float ry = b.mult / sqrtf(block_sum(ss, red) / (float)W + eps);
+        const float ry = b.w ? b.mult / sqrtf(block_sum(ss, red) / (float)W + eps) : b.mult;
 #pragma unroll
         for (int k = 0; k < NV; ++k) {
             const int c = (threadIdx.x + k * 256) * 4;
             if (c < W) {
-                FVec<4> g; g.load(b.w + c);
+                FVec<4> g;
+                if (b.w) g.load(b.w + c);
 #pragma unroll
-                for (int e = 0; e < 4; ++e) v[k].v[e] = fmaf(y[k].v[e] * ry, g.v[e], v[k].v[e]);
-                if (!rows) v[k].store(xr + c);
+                for (int e = 0; e < 4; ++e) v[k].v[e] = fmaf(y[k].v[e] * ry, b.w ? g.v[e] : 1.f, v[k].v[e]);
             }
         }
     }
+    if (b.add_rows || b.add_vec)
+#pragma unroll
+        for (int k = 0; k < NV; ++k) {
+            const int c = (threadIdx.x + k * 256) * 4;
+            if (c < W) { FVec<4> u = branch_add(b, src, W, c, v[k]); v[k] = u; }
+        }
+    if (!rows && (b.y || b.add_rows || b.add_vec))
+#pragma unroll
+        for (int k = 0; k < NV; ++k) { const int c = (threadIdx.x + k * 256) * 4; if (c < W) v[k].store(xr + c); }
     if (!w) return;
     float ss = 0.f;
 #pragma unroll
@@ -245,18 +270,23 @@ __global__ void __launch_bounds__(256) hy_branch_norm_kernel(float* __restrict__
     __shared__ float red[32];
     const long long t = blockIdx.x, src = rows ? rows[t] : t;
     float* xr = x + src * W;
-    float ry = 0.f;
-    if (b.y) {
+    float ry = b.mult;
+    if (b.y && b.w) {
         float ss = 0.f;
         for (int c = threadIdx.x; c < W; c += blockDim.x) { FVec<1> y; branch_load<1>(b, src, W, c, y); ss = fmaf(y.v[0], y.v[0], ss); }
         ry = b.mult / sqrtf(block_sum(ss, red) / (float)W + eps);
     }
-    auto value = [&](int c) { if (!b.y) return xr[c]; FVec<1> y; branch_load<1>(b, src, W, c, y); return fmaf(y.v[0] * ry, b.w[c], xr[c]); };
+    auto value = [&](int c) {
+        FVec<1> x, y; x.v[0] = xr[c];
+        if (b.y) { branch_load<1>(b, src, W, c, y); x.v[0] = fmaf(y.v[0] * ry, b.w ? b.w[c] : 1.f, x.v[0]); }
+        return branch_add<1>(b, src, W, c, x).v[0];
+    };
+    const bool store = !rows && (b.y || b.add_rows || b.add_vec);
     float ss = 0.f;
     for (int c = threadIdx.x; c < W; c += blockDim.x) {
         const float v = value(c);
         ss = fmaf(v, v, ss);
-        if (!rows && b.y) xr[c] = v;                 // a thread reads again only what it alone has written
+        if (store) xr[c] = v;                        // a thread reads again only what it alone has written
     }
     if (!w) return;
     const float rr = 1.0f / sqrtf(block_sum(ss, red) / (float)W + eps);
@@ -317,7 +347,7 @@ template <typename TA>
 cudaError_t branch_norm_t(float* x, const HyBranch& b, const int32_t* rows, const float* w, float eps, void* h, int ldh, int T, int W, cudaStream_t s) {
     auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
     // the form follows from the model's sizes alone, so a row takes the same kernel in every step
-    if (W % 4 == 0 && W <= 8192 && ldh % 4 == 0 && al16(x) && al16(b.y) && al16(b.w) && al16(w) && al16(h)) {
+    if (W % 4 == 0 && W <= 8192 && ldh % 4 == 0 && al16(x) && al16(b.y) && al16(b.w) && al16(b.add_rows) && al16(b.add_vec) && al16(w) && al16(h)) {
         if (W <= 1024) return launch_plain(hy_branch_norm_reg_kernel<TA, 1>, dim3(T), dim3(256), 0, s, x, b, rows, w, eps, (TA*)h, ldh, W);
         if (W <= 2048) return launch_plain(hy_branch_norm_reg_kernel<TA, 2>, dim3(T), dim3(256), 0, s, x, b, rows, w, eps, (TA*)h, ldh, W);
         if (W <= 4096) return launch_plain(hy_branch_norm_reg_kernel<TA, 4>, dim3(T), dim3(256), 0, s, x, b, rows, w, eps, (TA*)h, ldh, W);

@@ -97,13 +97,14 @@ __global__ void __launch_bounds__(128) hy_win_prep_vec8_kernel(HyWinAttn a, __nv
 }
 
 // qk_norm = 2: one RMS norm over the whole q projection of the row (all heads and maps) and one over the whole k projection, weights of
-// those sizes; then the query temperature.  Queries in place, keys and values into the row's cache slot.  One CTA per row.
+// those sizes; then the query temperature and the rotary (rot.dims > 0).  Queries in place, keys and values into the row's cache slot.  One CTA per row.
 __device__ __forceinline__ float win_q_temp(const HyWinAttn& a, int pos) {
     return a.q_temp_every > 0 ? 1.0f + a.q_temp_coef * logf((float)((pos + 1) / a.q_temp_every) + 1.0f) : 1.0f;
 }
 template <typename TA>
 __global__ void __launch_bounds__(128) hy_win_prep_whole_kernel(HyWinAttn a, TA* __restrict__ q, int ldq, const TA* __restrict__ k, const TA* __restrict__ v, int ldkv,
-                                                                const float* __restrict__ qw, const float* __restrict__ kw, float eps, TA* __restrict__ cache, HyRows r) {
+                                                                const float* __restrict__ qw, const float* __restrict__ kw, float eps, TA* __restrict__ cache, HyRows r,
+                                                                HyRotary rot) {
     HY_PDL();
     __shared__ float red[32];
     const long long t = blockIdx.x;
@@ -114,8 +115,19 @@ __global__ void __launch_bounds__(128) hy_win_prep_whole_kernel(HyWinAttn a, TA*
     if (k) for (int c = threadIdx.x; c < KW; c += blockDim.x) { const float x = ldf(k + t * ldkv + c); sk = fmaf(x, x, sk); }
     const float rq = 1.0f / sqrtf(block_sum(sq, red) / (float)QW + eps) * win_q_temp(a, r.positions[t]);
     const float rk = k ? 1.0f / sqrtf(block_sum(sk, red) / (float)KW + eps) : 0.f;
-    for (int c = threadIdx.x; c < QW; c += blockDim.x) stf(qr + c, ldf(qr + c) * rq * qw[c]);
-    if (k) for (int c = threadIdx.x; c < KW; c += blockDim.x) stf(crow + c, ldf(k + t * ldkv + c) * rk * kw[c]);
+    // work items of a head: the rotated pairs (one thread turns both channels), then the other channels one by one
+    const int half = rot.dims / 2, per = half + (a.dim - rot.dims);
+    const float* cs = rot.cos + (long long)r.positions[t] * half; const float* sn = rot.sin + (long long)r.positions[t] * half;
+    auto finish = [&](const TA* src, TA* dst, const float* w, float rr, int i) {
+        const int h0 = i / per * a.dim, j = i % per;
+        if (j < half) {
+            const int c0 = h0 + (rot.layout ? j : 2 * j), c1 = h0 + (rot.layout ? j + half : 2 * j + 1);
+            const float u = ldf(src + c0) * rr * w[c0], x = ldf(src + c1) * rr * w[c1];
+            stf(dst + c0, u * cs[j] - x * sn[j]); stf(dst + c1, x * cs[j] + u * sn[j]);
+        } else { const int c = h0 + rot.dims + (j - half); stf(dst + c, ldf(src + c) * rr * w[c]); }
+    };
+    for (int i = threadIdx.x; i < a.heads * a.maps * per; i += blockDim.x) finish(qr, qr, qw, rq, i);
+    if (k) for (int i = threadIdx.x; i < a.kv_heads * a.maps * per; i += blockDim.x) finish(k + t * ldkv, crow, kw, rk, i);
     if (v) for (int c = threadIdx.x; c < a.kv_heads * a.vdim; c += blockDim.x) crow[KW + c] = v[t * ldkv + c];
 }
 
@@ -124,7 +136,7 @@ __global__ void __launch_bounds__(128) hy_win_prep_whole_kernel(HyWinAttn a, TA*
 // last fp32 bits only; a model takes one of the two for all of its steps.
 __global__ void __launch_bounds__(128) hy_win_prep_whole_vec8_kernel(HyWinAttn a, __nv_bfloat16* __restrict__ q, int ldq, const __nv_bfloat16* __restrict__ k,
                                                                      const __nv_bfloat16* __restrict__ v, int ldkv, const float* __restrict__ qw, const float* __restrict__ kw, float eps,
-                                                                     __nv_bfloat16* __restrict__ cache, HyRows r) {
+                                                                     __nv_bfloat16* __restrict__ cache, HyRows r, HyRotary rot) {
     HY_PDL();
     __shared__ float red[32];
     const long long t = blockIdx.x;
@@ -147,8 +159,27 @@ __global__ void __launch_bounds__(128) hy_win_prep_whole_vec8_kernel(HyWinAttn a
     if (k) for (int c = threadIdx.x * 8; c < KW; c += blockDim.x * 8) sk += sq8(*reinterpret_cast<const uint4*>(k + t * ldkv + c));
     const float rq = 1.0f / sqrtf(block_sum(sq, red) / (float)QW + eps) * win_q_temp(a, r.positions[t]);
     const float rk = k ? 1.0f / sqrtf(block_sum(sk, red) / (float)KW + eps) : 0.f;
-    for (int c = threadIdx.x * 8; c < QW; c += blockDim.x * 8) *reinterpret_cast<uint4*>(qr + c) = scale8(*reinterpret_cast<const uint4*>(qr + c), rq, qw + c);
-    if (k) for (int c = threadIdx.x * 8; c < KW; c += blockDim.x * 8) *reinterpret_cast<uint4*>(crow + c) = scale8(*reinterpret_cast<const uint4*>(k + t * ldkv + c), rk, kw + c);
+    // rotated channels: the thread of a group of 8 in a head's first half turns its partner group too (rotate-half pairs, rot.dims / 2 a multiple of 8)
+    const int half = rot.dims / 2;
+    const float* cs = rot.cos + (long long)r.positions[t] * half; const float* sn = rot.sin + (long long)r.positions[t] * half;
+    auto norm8 = [](const uint4& u, float rr, const float* w, float* f) {
+        const float4 w0 = *reinterpret_cast<const float4*>(w), w1 = *reinterpret_cast<const float4*>(w + 4);
+        f[0] = bf16lo(u.x) * rr * w0.x; f[1] = bf16hi(u.x) * rr * w0.y; f[2] = bf16lo(u.y) * rr * w0.z; f[3] = bf16hi(u.y) * rr * w0.w;
+        f[4] = bf16lo(u.z) * rr * w1.x; f[5] = bf16hi(u.z) * rr * w1.y; f[6] = bf16lo(u.w) * rr * w1.z; f[7] = bf16hi(u.w) * rr * w1.w;
+    };
+    auto finish = [&](const __nv_bfloat16* src, __nv_bfloat16* dst, const float* w, float rr, int c) {
+        const int d = rot.dims > 0 ? c % a.dim : 0;
+        if (rot.dims == 0 || d >= rot.dims) { *reinterpret_cast<uint4*>(dst + c) = scale8(*reinterpret_cast<const uint4*>(src + c), rr, w + c); return; }
+        if (d >= half) return;
+        float u[8], x[8], o[8], p[8];
+        norm8(*reinterpret_cast<const uint4*>(src + c), rr, w + c, u); norm8(*reinterpret_cast<const uint4*>(src + c + half), rr, w + c + half, x);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) { const float co = cs[d + e], si = sn[d + e]; o[e] = u[e] * co - x[e] * si; p[e] = x[e] * co + u[e] * si; }
+        *reinterpret_cast<uint4*>(dst + c) = make_uint4(pack_bf16x2(o[0], o[1]), pack_bf16x2(o[2], o[3]), pack_bf16x2(o[4], o[5]), pack_bf16x2(o[6], o[7]));
+        *reinterpret_cast<uint4*>(dst + c + half) = make_uint4(pack_bf16x2(p[0], p[1]), pack_bf16x2(p[2], p[3]), pack_bf16x2(p[4], p[5]), pack_bf16x2(p[6], p[7]));
+    };
+    for (int c = threadIdx.x * 8; c < QW; c += blockDim.x * 8) finish(qr, qr, qw, rq, c);
+    if (k) for (int c = threadIdx.x * 8; c < KW; c += blockDim.x * 8) finish(k + t * ldkv, crow, kw, rk, c);
     if (v) for (int c = threadIdx.x * 8; c < VW; c += blockDim.x * 8) *reinterpret_cast<uint4*>(crow + KW + c) = *reinterpret_cast<const uint4*>(v + t * ldkv + c);
 }
 
@@ -927,16 +958,19 @@ cudaError_t hy_rmsnorm_pair(bool f32, const float* x, const int32_t* rows, const
 }
 
 cudaError_t hy_win_prep(bool f32, const HyWinAttn& a, void* q, int ldq, const void* k, const void* v, int ldkv, const float* q_norm_w, const float* k_norm_w, float eps, void* cache,
-                        const HyRows& r, cudaStream_t s) {
+                        const HyRows& r, cudaStream_t s, const HyRotary* rotary) {
     if (r.T <= 0 || (!a.qk_norm && !k && a.q_temp_every <= 0)) return cudaSuccess;
     using bf = __nv_bfloat16;
-    if (a.qk_norm == 2 && !f32 && (a.heads * a.maps * a.dim) % 8 == 0 && (a.kv_heads * a.maps * a.dim) % 8 == 0 && (a.kv_heads * a.vdim) % 8 == 0 && ldq % 8 == 0 && ldkv % 8 == 0 &&
+    const HyRotary rot = rotary ? *rotary : HyRotary{0, 0, nullptr, nullptr, nullptr, nullptr};
+    if (rot.dims > 0 && (a.qk_norm != 2 || (rot.dims & 1) || rot.dims > a.dim || rot.v_cos)) return cudaErrorInvalidValue;      // the rotary rides in the whole-projection form only
+    const bool rot8 = rot.dims == 0 || (rot.layout == 1 && rot.dims % 16 == 0 && a.dim % 8 == 0);
+    if (a.qk_norm == 2 && !f32 && rot8 && (a.heads * a.maps * a.dim) % 8 == 0 && (a.kv_heads * a.maps * a.dim) % 8 == 0 && (a.kv_heads * a.vdim) % 8 == 0 && ldq % 8 == 0 && ldkv % 8 == 0 &&
         ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v) | reinterpret_cast<uintptr_t>(cache) | reinterpret_cast<uintptr_t>(q_norm_w) |
           reinterpret_cast<uintptr_t>(k_norm_w)) & 15) == 0)
-        return launch_plain(hy_win_prep_whole_vec8_kernel, dim3(r.T), dim3(128), 0, s, a, (bf*)q, ldq, (const bf*)k, (const bf*)v, ldkv, q_norm_w, k_norm_w, eps, (bf*)cache, r);
+        return launch_plain(hy_win_prep_whole_vec8_kernel, dim3(r.T), dim3(128), 0, s, a, (bf*)q, ldq, (const bf*)k, (const bf*)v, ldkv, q_norm_w, k_norm_w, eps, (bf*)cache, r, rot);
     if (a.qk_norm == 2)
-        return f32 ? launch_plain(hy_win_prep_whole_kernel<float>, dim3(r.T), dim3(128), 0, s, a, (float*)q, ldq, (const float*)k, (const float*)v, ldkv, q_norm_w, k_norm_w, eps, (float*)cache, r)
-                   : launch_plain(hy_win_prep_whole_kernel<bf>, dim3(r.T), dim3(128), 0, s, a, (bf*)q, ldq, (const bf*)k, (const bf*)v, ldkv, q_norm_w, k_norm_w, eps, (bf*)cache, r);
+        return f32 ? launch_plain(hy_win_prep_whole_kernel<float>, dim3(r.T), dim3(128), 0, s, a, (float*)q, ldq, (const float*)k, (const float*)v, ldkv, q_norm_w, k_norm_w, eps, (float*)cache, r, rot)
+                   : launch_plain(hy_win_prep_whole_kernel<bf>, dim3(r.T), dim3(128), 0, s, a, (bf*)q, ldq, (const bf*)k, (const bf*)v, ldkv, q_norm_w, k_norm_w, eps, (bf*)cache, r, rot);
     if (a.q_temp_every > 0) return cudaErrorInvalidValue;      // the query temperature is applied by the whole-projection form only
     const int gs = a.dim / 8;
     const bool aligned = ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v) | reinterpret_cast<uintptr_t>(cache) |
@@ -1010,7 +1044,7 @@ cudaError_t hy_win_attention(bool f32, const HyWinAttn& a, const void* q, int ld
 
 static bool win_modded(const HyWinAttn& a) { return a.softcap > 0.f || a.slope_exp > 0.f; }
 bool hy_win_mma_supported(const HyWinAttn& a) {
-    const bool vd_ok = a.vdim == 16 || a.vdim == 32 || a.vdim == 64 || a.vdim == 96 || a.vdim == 128 || (a.rel && (a.vdim == 48 || a.vdim == 80));
+    const bool vd_ok = a.vdim == 16 || a.vdim == 32 || a.vdim == 64 || a.vdim == 96 || a.vdim == 128 || ((a.rel || win_modded(a)) && (a.vdim == 48 || a.vdim == 80));
     return hy_win_supported(a) && a.dim % 16 == 0 && a.dim <= 128 && vd_ok && !((win_modded(a) || a.rel) && a.maps != 1) && !(win_modded(a) && a.rel) && a.out_rot != 2;      // score modifiers on the tensor cores: one map; outputs turned back in pairs of neighbours only
 }
 template <int MAPS, int NVB, int MOD>
@@ -1050,7 +1084,7 @@ cudaError_t hy_win_attention_mma(const HyWinAttn& a, const void* q, int ldq, con
     if (!hy_win_mma_supported(a)) return cudaErrorInvalidValue;
 #define WIN_CASE(M, N) if (a.maps == M && a.vdim == N * 8) return win_mma_launch<M, N, WIN_MOD_NONE>(a, q, ldq, cache, sink, gate, ldg, out, ldo, eps, r, tile_seq, tile_q0, n_tiles, s)
 #define WIN_CASE_MOD(N) if (a.vdim == N * 8) return win_mma_launch<1, N, WIN_MOD_CAP_SLOPE>(a, q, ldq, cache, sink, gate, ldg, out, ldo, eps, r, tile_seq, tile_q0, n_tiles, s)
-    if (win_modded(a)) { WIN_CASE_MOD(2); WIN_CASE_MOD(4); WIN_CASE_MOD(8); WIN_CASE_MOD(12); WIN_CASE_MOD(16); return cudaErrorInvalidValue; }
+    if (win_modded(a)) { WIN_CASE_MOD(2); WIN_CASE_MOD(4); WIN_CASE_MOD(6); WIN_CASE_MOD(8); WIN_CASE_MOD(10); WIN_CASE_MOD(12); WIN_CASE_MOD(16); return cudaErrorInvalidValue; }
 #define WIN_CASE_REL(N) if (a.vdim == N * 8) return win_mma_launch<1, N, WIN_MOD_REL>(a, q, ldq, cache, sink, gate, ldg, out, ldo, eps, r, tile_seq, tile_q0, n_tiles, s)
     if (a.rel) { WIN_CASE_REL(2); WIN_CASE_REL(4); WIN_CASE_REL(6); WIN_CASE_REL(8); WIN_CASE_REL(10); WIN_CASE_REL(12); WIN_CASE_REL(16); return cudaErrorInvalidValue; }
     WIN_CASE(1, 2); WIN_CASE(1, 4); WIN_CASE(1, 8); WIN_CASE(1, 12); WIN_CASE(1, 16);
@@ -1066,7 +1100,7 @@ cudaError_t hy_win_decode_mma(const HyWinAttn& a, const void* q, int ldq, const 
     if (!hy_win_mma_supported(a)) return cudaErrorInvalidValue;
 #define WIN_CASE(M, N) if (a.maps == M && a.vdim == N * 8) return win_decode_launch<M, N, WIN_MOD_NONE>(a, q, ldq, cache, sink, gate, ldg, out, ldo, eps, r, tile_seq, tile_q0, n_tiles, s)
 #define WIN_CASE_MOD(N) if (a.vdim == N * 8) return win_decode_launch<1, N, WIN_MOD_CAP_SLOPE>(a, q, ldq, cache, sink, gate, ldg, out, ldo, eps, r, tile_seq, tile_q0, n_tiles, s)
-    if (win_modded(a)) { WIN_CASE_MOD(2); WIN_CASE_MOD(4); WIN_CASE_MOD(8); WIN_CASE_MOD(12); WIN_CASE_MOD(16); return cudaErrorInvalidValue; }
+    if (win_modded(a)) { WIN_CASE_MOD(2); WIN_CASE_MOD(4); WIN_CASE_MOD(6); WIN_CASE_MOD(8); WIN_CASE_MOD(10); WIN_CASE_MOD(12); WIN_CASE_MOD(16); return cudaErrorInvalidValue; }
 #define WIN_CASE_REL(N) if (a.vdim == N * 8) return win_decode_launch<1, N, WIN_MOD_REL>(a, q, ldq, cache, sink, gate, ldg, out, ldo, eps, r, tile_seq, tile_q0, n_tiles, s)
     if (a.rel) { WIN_CASE_REL(2); WIN_CASE_REL(4); WIN_CASE_REL(6); WIN_CASE_REL(8); WIN_CASE_REL(10); WIN_CASE_REL(12); WIN_CASE_REL(16); return cudaErrorInvalidValue; }
     WIN_CASE(1, 2); WIN_CASE(1, 4); WIN_CASE(1, 8); WIN_CASE(1, 12); WIN_CASE(1, 16);

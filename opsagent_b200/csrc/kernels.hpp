@@ -16,9 +16,9 @@ int make_tmap_bf16_2d(CUtensorMap* out, const void* base, uint64_t rows, uint64_
 
 // ---- GEMM (gemm_tcgen05.cu): C[M,N] = A[M,K] . B[N,K]^T, bf16 in, fp32 accumulate in TMEM -------
 enum GemmEpilogue : int {
-    EPI_STORE = 0,    // out[M,N] bf16 = act(acc (+ bias[N])), act = identity, relu(.)^2 or the tanh form of GELU (GemmParams::store_act)
+    EPI_STORE = 0,    // out[M,N] bf16 = act(acc (+ bias[N])), act = identity, relu(.)^2, the tanh form of GELU, or SiLU on a range of columns (GemmParams::store_act)
     EPI_RESID = 1,    // out[M,N] bf16 = acc + resid[M,N]      (out may alias resid)
-    EPI_SWIGLU = 2,   // out[M,N/2] bf16 = silu(gate)*up, B rows interleaved 16 gate / 16 up; GemmParams::glu_limit > 0: the clamped gated activation, rows scaled before it
+    EPI_SWIGLU = 2,   // out[M,N/2] bf16 = silu(gate)*up (GemmParams::glu_gelu: gelu_tanh(gate)*up), B rows interleaved 16 gate / 16 up; GemmParams::glu_limit > 0: the clamped gated activation, rows scaled before it
     EPI_LOGITS = 3,   // per-row (max, argmax) partial per N-tile -> argmax_ws; optional fp32 logits store
     EPI_F32 = 4,      // f32_out[M,N] fp32 = alpha * acc (+ bias_f32[N]) (+ f32_out when f32_accumulate): fp32 residual streams and logits
 };
@@ -26,7 +26,8 @@ struct GemmParams {
     int M, N, K;
     void* out; int ldo;             // bf16 output, leading dimension in elements
     const void* bias;               // bf16 [N] or null        (EPI_STORE)
-    int store_act;                  // EPI_STORE: 0 = store as is, 1 = relu(.)^2 (gate-less experts' activation), 2 = gelu_tanh(.) (dense feed-forward)
+    int store_act;                  // EPI_STORE: 0 = store as is, 1 = relu(.)^2 (gate-less experts' activation), 2 = gelu_tanh(.) (dense feed-forward), 3 = silu(.) on columns act_col0 .. act_col1 - 1 (multiples of 8), the others as they are
+    int act_col0, act_col1;
     const void* resid; int ldr;     // bf16 [M, ldr]           (EPI_RESID)
     float* logits; int ldl;         // optional fp32 [M, ldl]  (EPI_LOGITS)
     float* amax_val; int* amax_idx; // [M, n_tiles]            (EPI_LOGITS)
@@ -40,6 +41,7 @@ struct GemmParams {
     // EPI_SWIGLU with glu_limit > 0: out = g sigmoid(glu_slope g) (u + 1), g = min(s gate, limit), u = clamp(s up, -limit, limit), where row r's s is
     // row_scale[row_scale_idx[r]] (0 for a negative index: a padding row of a grouped product) — the router's weight on an expert's input, exact in fp32
     float glu_limit, glu_slope; const float* row_scale; const int32_t* row_scale_idx;
+    int glu_gelu;                   // EPI_SWIGLU: the gate passes the tanh form of GELU instead of SiLU
 };
 // tmA: box {64, 128} over A[M,K]; tmB: box {64, block_n} over B[N,K].  block_n in {32,64,128,256}.
 cudaError_t launch_gemm(const CUtensorMap* tmA, const CUtensorMap* tmB, const GemmParams& p, int epilogue, int block_n,

@@ -1,9 +1,10 @@
-"""Throughput of the hybrid family beside the closest existing models (`bench.py --arch ratasun | zurevik | rofizen | gosavik | petipel`): Ratasun beside the
+"""Throughput of the hybrid family beside the closest existing models (`bench.py --arch ratasun | zurevik | rofizen | gosavik | petipel | ketopel`): Ratasun beside the
 Llama-family model of equal width, depth and active feed-forward size; Zurevik and Rofizen beside the Ratasun model of equal width, depth and
 experts (the closest design: routed experts in every layer; recurrent mixers with an fp32 state like Rofizen's) and beside that Llama-family model;
 Gosavik (dense feed-forward, attention mixers only) beside the Llama-family model of equal width, depth and feed-forward size — the closest model as a whole —
 and beside Ratasun, whose latent attention is the closest kernel to its own; Petipel (linear attention with a gate per key channel, cached-key/value
-attention, routed experts) beside Rofizen, which has the closest kernel for each of its own, and beside both of those.  Random weights (seeded on load), synthetic token ids; prefill = real chunked prefill of batch x (ctx-1) tokens,
+attention, routed experts) beside Rofizen, which has the closest kernel for each of its own, and beside both of those; Ketopel beside Ratasun (delta rule, latent attention), Rofizen (capped attention beside a
+linear recurrence) and the Llama-family model (gated feed-forward) of equal width, depth and sizes.  Random weights (seeded on load), synthetic token ids; prefill = real chunked prefill of batch x (ctx-1) tokens,
 decode = steps of the whole batch, both timed with CUDA events inside the engine (oa_bench_decode).  With --breakdown the per-kernel-class
 device times come from the engine's in-situ event timing (OA_PROFILE_ALL), one pass for prefill and one for decode."""
 from __future__ import annotations
@@ -106,6 +107,30 @@ def petipel_sizes(name: str) -> dict:
             "layers": [{"type": t, "mixer": m, "mlp": f} for t, m, f in [("hgrn2", rec, dense), ("attention", att, moe)] * 3]}
 
 
+def ketopel_sizes(name: str) -> dict:
+    """Ketopel at the width and depth (6 layer executions: [delta rule, capped attention beside lightning attention] twice with the same weights, then
+    latent attention, delta rule) of sizes(name), the mixers at the sizes of Ratasun's and Rofizen's, the gated feed-forward at the Llama case's."""
+    if name == "small":
+        dl = {"heads": 8, "kv_heads": 4, "dim": 64, "vdim": 128, "conv": 4}
+        left = {"heads": 16, "kv_heads": 4, "dim": 64, "vdim": 64, "scale": 64 ** -0.5}
+        right = {"heads": 8, "dim": 64, "vdim": 128}
+        lat = {"heads": 16, "dim": 64, "rot_dim": 32, "vdim": 64, "kv_rank": 256, "scale": 96 ** -0.5, "rot": {"base": 10000.0, "dims": 32}}
+        width, ff = 1024, 2048
+    else:
+        dl = {"heads": 16, "kv_heads": 8, "dim": 128, "vdim": 128, "conv": 4}
+        left = {"heads": 16, "kv_heads": 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
+        right = {"heads": 16, "dim": 128, "vdim": 128}
+        lat = {"heads": 16, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": 192 ** -0.5, "rot": {"base": 10000.0, "dims": 64}}
+        width, ff = 2048, 4096
+    left.update(softcap=30.0, rot={"base": 1000000.0, "dims": left["dim"] // 2, "scaling": {"factor": 4.0, "original": 2048, "fast": 24.0, "slow": 2.0}})
+    right["decay"] = [1.0 - 2.0 ** (-1 - 9 * h / right["heads"]) for h in range(right["heads"])]
+    par = {"left": left, "right": right, "left_scale": 0.8, "right_scale": 0.6}
+    mlp = {"kind": "dense", "ff": ff}
+    order = [("delta", dl), ("parallel", par), ("latent_attention", lat), ("delta", dl)]
+    return {"architecture": "Ketopel", "width": width, "vocab": 32000, "norm": {"eps": 1e-6}, "embedding": {"scale": 2.0}, "loop": {"start": 0, "stop": 2, "times": 2},
+            "layers": [{"type": t, "mixer": m, "mlp": mlp} for t, m in order]}
+
+
 def one(engine_cfg: dict, batch: int, ctx: int, steps: int, warmup: int, breakdown: bool) -> dict:
     from .engine import Engine
     out = {}
@@ -131,7 +156,7 @@ def one(engine_cfg: dict, batch: int, ctx: int, steps: int, warmup: int, breakdo
 
 
 def run(args) -> None:
-    zu = args.arch in ("zurevik", "rofizen", "gosavik", "petipel")
+    zu = args.arch in ("zurevik", "rofizen", "gosavik", "petipel", "ketopel")
     res = {"metric": args.arch + "_vs_ratasun_and_llama_throughput" if zu else "hybrid_vs_llama_throughput", "unit": "tokens/s", "data": "synthetic", "dtype": "bf16", "cases": []}
     for name in args.arch_sizes.split(","):
         sz = sizes(name)
@@ -146,15 +171,15 @@ def run(args) -> None:
                 return one(dict(common, model_dir=d, **json.loads(args.engine_extra)), batch, ctx, args.steps, args.warmup, args.breakdown)
         case = {"size": name, "batch": batch, "ctx": ctx, "layer_runs": sz["runs"]}
         if zu:
-            case[args.arch] = folder_model({"zurevik": zurevik_sizes, "rofizen": rofizen_sizes, "gosavik": gosavik_sizes, "petipel": petipel_sizes}[args.arch](name))
-        if args.arch == "petipel":
+            case[args.arch] = folder_model({"zurevik": zurevik_sizes, "rofizen": rofizen_sizes, "gosavik": gosavik_sizes, "petipel": petipel_sizes, "ketopel": ketopel_sizes}[args.arch](name))
+        if args.arch in ("petipel", "ketopel"):
             case["rofizen"] = folder_model(rofizen_sizes(name))
         case["ratasun"] = hy = folder_model(sz["hybrid"])
         case["llama_equal_size"] = ll = one(dict(common, **sz["llama"]), batch, ctx, args.steps, args.warmup, args.breakdown)
         new = case[args.arch] if zu else hy
         case["prefill_ratio"], case["decode_ratio"] = new["prefill_tok_s"] / ll["prefill_tok_s"], new["decode_tok_s"] / ll["decode_tok_s"]
         if zu:
-            if args.arch == "petipel":
+            if args.arch in ("petipel", "ketopel"):
                 case["prefill_ratio_to_rofizen"], case["decode_ratio_to_rofizen"] = (new[k] / case["rofizen"][k] for k in ("prefill_tok_s", "decode_tok_s"))
             case["prefill_ratio_to_ratasun"], case["decode_ratio_to_ratasun"] = new["prefill_tok_s"] / hy["prefill_tok_s"], new["decode_tok_s"] / hy["decode_tok_s"]
         res["cases"].append(case)

@@ -942,6 +942,37 @@ __global__ void __launch_bounds__(128) hy_gated_norm_warp_kernel(const float* __
     }
 }
 
+// Groups too wide for a warp (gate behind the norm, or none): one CTA per (row, group), the group's values in registers, 16-byte accesses
+template <typename TA, int NV>      // NV x 4 channels per thread: group <= 1024 NV
+__global__ void __launch_bounds__(256) hy_gated_norm_wide_kernel(const float* __restrict__ o, int C, int group, const float* __restrict__ w, int wlen, const TA* __restrict__ gate, int ld_gate, int act,
+                                                                 TA* __restrict__ out, int ld_out, float eps) {
+    HY_PDL();
+    __shared__ float red[32];
+    const long long t = blockIdx.x; const int c0 = blockIdx.y * group;
+    float v[NV][4], g[NV][4], ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int i = (threadIdx.x + k * 256) * 4;
+        if (i < group) {
+            ld4(o + t * C + c0 + i, v[k]);
+            if (gate) ld4(gate + t * ld_gate + c0 + i, g[k]);
+            ss += (v[k][0] * v[k][0] + v[k][1] * v[k][1]) + (v[k][2] * v[k][2] + v[k][3] * v[k][3]);
+        }
+    }
+    const float rr = 1.0f / sqrtf(block_sum(ss, red) / (float)group + eps);
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int i = (threadIdx.x + k * 256) * 4;
+        if (i >= group) continue;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            v[k][e] *= rr * (w ? w[(c0 + i + e) % wlen] : 1.f);
+            if (gate) v[k][e] *= act ? siluf_(g[k][e]) : sigmoidf_(g[k][e]);
+        }
+        st4(out + t * ld_out + c0 + i, v[k]);
+    }
+}
+
 // ---------------------------------------------------------------------------------------------------------------------------------
 // mixture of experts
 // ---------------------------------------------------------------------------------------------------------------------------------
@@ -1413,6 +1444,12 @@ cudaError_t hy_gated_norm(bool f32, const float* o, int C, int group, const floa
                    : launch_plain(hy_gated_norm_warp_kernel<bf>, g, dim3(128), 0, s, o, C, group, w, wlen, (const bf*)gate, ld_gate, gate_before, act, skip, skip_block, (const bf*)xs, ld_xs, (bf*)out, ld_out, eps, n, den_dot, den_floor);
     }
     dim3 grid(T, C / group);
+    if (group % 4 == 0 && group > 512 && group <= 8192 && !skip && !den_dot && !(gate && gate_before) && C % 4 == 0 && ld_gate % 4 == 0 && ld_out % 4 == 0 && al(o, 16) && al(gate, 4 * ea) && al(out, 4 * ea)) {
+#define HY_GNW(NV) (f32 ? launch_plain(hy_gated_norm_wide_kernel<float, NV>, grid, dim3(256), 0, s, o, C, group, w, wlen, (const float*)gate, ld_gate, act, (float*)out, ld_out, eps) \
+                        : launch_plain(hy_gated_norm_wide_kernel<bf, NV>, grid, dim3(256), 0, s, o, C, group, w, wlen, (const bf*)gate, ld_gate, act, (bf*)out, ld_out, eps))
+        return group <= 1024 ? HY_GNW(1) : group <= 2048 ? HY_GNW(2) : group <= 4096 ? HY_GNW(4) : HY_GNW(8);
+#undef HY_GNW
+    }
     return f32 ? launch_plain(hy_gated_norm_kernel<float>, grid, dim3(128), 0, s, o, C, group, w, wlen, (const float*)gate, ld_gate, gate_before, act, skip, skip_block, (const float*)xs, ld_xs, (float*)out, ld_out, eps, den_dot, den_floor)
                : launch_plain(hy_gated_norm_kernel<bf>, grid, dim3(128), 0, s, o, C, group, w, wlen, (const bf*)gate, ld_gate, gate_before, act, skip, skip_block, (const bf*)xs, ld_xs, (bf*)out, ld_out, eps, den_dot, den_floor);
 }

@@ -203,6 +203,21 @@ constexpr int HY_FORGET_FEW_ROWS = 4;
 bool hy_forget_mix_supported(int dim, int vdim);        // multiples of 8 up to 128
 cudaError_t hy_forget_mix(int heads, int dim, int vdim, const void* q, const void* z, const void* v, int ld, const float* bias, const float* lower, const float* norm_w, float eps, float* state,
                           void* out, int ldo, bool few, bool many, const HyRows& r, cudaStream_t s);
+// The recurrences with one decay per head between their projections, bf16 (sizes below), in two forms picked per sequence: token by token where it
+// brings at most HY_FORGET_FEW_ROWS rows to the step, blocks of 32 tokens on the tensor cores where it brings more; the fp32 state stays on chip for
+// the whole portion.  few / many: whether the step has sequences of either kind.
+bool hy_block_memory_supported(int dim, int vdim);        // multiples of 8 up to 128
+struct HyBlockHead { int heads, qk_heads, dim, vdim; };
+// Lightning attention: q, k, v [T, ld] (activated; qk_heads = heads): S <- decay_h S + k v^T, o = S^T q; out [T, heads vdim] fp32
+cudaError_t hy_lightning_mix(const HyBlockHead& m, const void* q, const void* k, const void* v, int ld, const float* decay, float* state, float* out, bool few, bool many, const HyRows& r,
+                             cudaStream_t s);
+// Gated delta rule with one decay per head: unit-norm q (times dim^-1/2) and k, S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q, RMS norm per head with the
+// weight norm_w [vdim], times silu(gate).  conv [T, ld_conv] = the activated short convolutions' rows [q heads | k heads | v heads] (read for `many` sequences); the rows of
+// `few` sequences go through the convolution here, from its inputs in [T, ld_in] (same columns), taps conv_w [channels, taps] and the carried tails.
+// a, b, gate: projections [T, ld_in]; out [T, ldo] bf16
+struct HyDeltaMix { const void* conv; int ld_conv; const void* in; int ld_in; const float* conv_w; int taps; const void* tails; const void* a; const void* b; const void* gate;
+                    const float* A_log; const float* dt_bias; const float* norm_w; float eps; };
+cudaError_t hy_delta_mix(const HyBlockHead& m, const HyDeltaMix& d, float* state, void* out, int ldo, bool few, bool many, const HyRows& r, cudaStream_t s);
 // Matrix memory.  gates [T, ldg] fp32 = [W_i h + b_i | W_f h + b_f] (heads each).  hy_mlstm_gates: log gates i = cap tanh(. / cap),
 // f = logsigmoid(cap tanh(. / cap)); the running maximum m_t = max(f_t + m_(t-1), i_t) per (sequence, head), carried in mstate [slots, heads]
 // (a sequence whose step starts at position 0 starts from m = 0); out: dec[t, h] = exp(f + m_(t-1) - m_t), gin[t, h] = exp(i - m_t), floor_[t, h] = exp(-m_t)

@@ -150,16 +150,6 @@ __global__ void __launch_bounds__(128) hy_lin_prep_kernel(HyLinPrep p, const TA*
 // The same for bf16 rows whose heads come in aligned groups of 8 channels (dim, vdim, rot_dims / 2 multiples of 8): a thread owns 8 channels,
 // every access is 16 bytes wide.  k_gate (matrix memory): k is multiplied by k_gate[t, head].  Per element the arithmetic is that of the
 // kernels above and below: the same bits.
-__device__ __forceinline__ void unpack8(const uint4& r, float* f) {
-    f[0] = bf16lo(r.x); f[1] = bf16hi(r.x); f[2] = bf16lo(r.y); f[3] = bf16hi(r.y); f[4] = bf16lo(r.z); f[5] = bf16hi(r.z); f[6] = bf16lo(r.w); f[7] = bf16hi(r.w);
-}
-__device__ __forceinline__ void ld8f(const float* p, float* f) {
-    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
-}
-__device__ __forceinline__ void st8f(float* p, const float* f) {
-    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]); *reinterpret_cast<float4*>(p + 4) = make_float4(f[4], f[5], f[6], f[7]);
-}
 __global__ void __launch_bounds__(128) hy_lin_prep_vec8_kernel(HyLinPrep p, const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k, const __nv_bfloat16* __restrict__ v,
                                                                int ld, float* __restrict__ qq, float* __restrict__ kk, float* __restrict__ vv, float* __restrict__ dec_channel,
                                                                float inv_tau, const float* __restrict__ decay_head, float* __restrict__ dec_head, const float* __restrict__ rope_cos,
@@ -444,8 +434,6 @@ __global__ void __launch_bounds__(256, 2) hy_forget_mix_kernel(const __nv_bfloat
 // accumulator fragments, which are the A operand of O^T = S^T (q B)^T as they stand; S^T += V^T (w ...) accumulates into them.  Operands that
 // are not bfloat16 already (the state as read, q B, w times gates, A) enter as a bfloat16 value plus a bfloat16 remainder, so the products are
 // accurate to about 2^-16 of their size (q B is rounded like the projection it comes from); the state itself stays fp32.  Tokens beyond the portion's end count as gates of one that write nothing.
-__device__ __forceinline__ void split_bf16(float x, __nv_bfloat16& hi, __nv_bfloat16& lo) { hi = __float2bfloat16_rn(x); lo = __float2bfloat16_rn(x - __bfloat162float(hi)); }
-__device__ __forceinline__ void split_pack(float a, float b, uint32_t& hi, uint32_t& lo) { hi = pack_bf16x2(a, b); lo = pack_bf16x2(a - bf16lo(hi), b - bf16hi(hi)); }
 template <int CV> __device__ __forceinline__ void load_cv(const float* p, float* f) {
 #pragma unroll
     for (int e = 0; e < CV; e += 4) { const float4 x = *reinterpret_cast<const float4*>(p + e); f[e] = x.x; f[e + 1] = x.y; f[e + 2] = x.z; f[e + 3] = x.w; }

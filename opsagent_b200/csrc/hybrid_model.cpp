@@ -706,9 +706,13 @@ void HybridModel::linear_mixer(const HyRun& run, const HyLayer& l, const LayerW&
         cuda_check(hy_recurrence(HY_REC_CHANNEL, qq_, kk_, vv_, dec_, nullptr, rec_, st, H, H, D, VD, r, stream), "forget-gate recurrence"); MARK(8);
         cuda_check(hy_gated_norm(f32_, rec_, H * VD, VD, w.norm_w, VD, nullptr, 4, 0, 0, nullptr, 1, nullptr, 0, mix_, ld_mix_, hc_.eps, T, stream), "head norm"); MARK(9);
     } else if (n.kind == HY_LIN_HEAD_DECAY) {
-        const float* rc = w.rope >= 0 ? ropes_[w.rope].cos : nullptr; const float* rs = w.rope >= 0 ? ropes_[w.rope].sin : nullptr;
+        const float* rc = n.rot_dims > 0 ? ropes_[w.rope].cos : nullptr; const float* rs = n.rot_dims > 0 ? ropes_[w.rope].sin : nullptr;
+        if (!f32_ && opt.hy_tensor_core && n.norm == HY_LIN_NORM_JOINT && n.rot_dims == 0 && !n.q_scaled && !n.k_scaled && hy_block_memory_supported(D, VD)) {       // by the model's sizes alone
+            cuda_check(hy_lightning_mix(HyBlockHead{H, H, D, VD}, q, k, v, ld_proj_, w.decay, st, rec_, few_rows_, many_rows_, r, stream), "lightning attention"); MARK(8);
+        } else {
         cuda_check(hy_lin_prep(f32_, HyLinPrep{H, D, VD, n.q_scaled, n.k_scaled, n.rot_dims}, q, k, v, ld_proj_, qq_, kk_, vv_, nullptr, 1.f, w.decay, dec_, rc, rs, r, stream), "retention operands"); MARK(28);
         cuda_check(hy_recurrence(HY_REC_SCALAR, qq_, kk_, vv_, dec_, nullptr, rec_, st, H, H, D, VD, r, stream), "retention"); MARK(8);
+        }
         if (n.norm == HY_LIN_NORM_JOINT) {       // one norm over all heads; a layer that joins two mixers puts it behind the attention side's heads
             cuda_check(hy_gated_norm(f32_, rec_, H * VD, H * VD, w.norm_w, H * VD, g, ld_proj_, 0, n.gate_silu, nullptr, 1, nullptr, 0, at(mix_, w.off_mix2), ld_mix_, hc_.eps, T, stream), "joint norm"); MARK(9);
             return;
@@ -740,6 +744,14 @@ void HybridModel::delta_mixer(const HyRun& run, const HyLayer& l, const LayerW& 
     const int T = r.T;
     auto at = [&](void* base, size_t elems) -> void* { return reinterpret_cast<char*>(base) + elems * es_; };
     const HyDelta d{l.heads, l.kv_heads, l.dim, l.vdim, l.head_decay};
+    if (l.head_decay && !f32_ && opt.hy_tensor_core && hy_block_memory_supported(l.dim, l.vdim)) {       // by the model's sizes alone; hy_tensor_core = 0 takes the separate kernels
+        const void* in = at(proj_, w.off_a);
+        if (many_rows_) { cuda_check(hy_conv_silu(f32_, in, ld_proj_, w.conv_ch, w.conv_w, nullptr, l.conv, conv_, ld_conv_, tails_[run.state_idx], r, stream), "conv"); MARK(6); }
+        const HyDeltaMix dm{conv_, ld_conv_, in, ld_proj_, w.conv_w, l.conv, tails_[run.state_idx], at(proj_, w.off_c), at(proj_, w.off_b), at(proj_, w.off_d), w.A_log, w.dt_bias, w.norm_w, hc_.eps};
+        cuda_check(hy_delta_mix(HyBlockHead{l.heads, l.kv_heads, l.dim, l.vdim}, dm, states_[run.state_idx], mix_, ld_mix_, few_rows_, many_rows_, r, stream), "delta rule"); MARK(8);
+        cuda_check(hy_conv_tails(f32_, in, ld_proj_, w.conv_ch, l.conv, tails_[run.state_idx], r, stream), "conv tails"); MARK(6);
+        return;
+    }
     cuda_check(hy_conv_silu(f32_, at(proj_, w.off_a), ld_proj_, w.conv_ch, w.conv_w, nullptr, l.conv, conv_, ld_conv_, tails_[run.state_idx], r, stream), "conv");
     cuda_check(hy_conv_tails(f32_, at(proj_, w.off_a), ld_proj_, w.conv_ch, l.conv, tails_[run.state_idx], r, stream), "conv tails"); MARK(6);
     const void *a = at(proj_, w.off_c), *g = at(proj_, w.off_d); int ld_a = ld_proj_, ld_g = ld_proj_;

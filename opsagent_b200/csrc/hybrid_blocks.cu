@@ -36,20 +36,23 @@ struct BlockArgs {
     const float *A_log, *dt_bias, *norm_w, *decay; float eps;
     float* state; void* out; int ldo, H, QH, D, VD;
 };
-struct BlockSmem {          // offsets in bytes
-    int QP, VP8, OP, row_bytes, buf, os, ph, pl, mh, ml, lf, sc, total;
+constexpr int BM_PP = BM_TB + 8, BM_PM = BM_TB * BM_PP;      // pitch and size of a 32 x 32 matrix of bf16 operands
+struct BlockSmem {          // offsets in bytes: three buffers of rows, read-outs, two sets of block matrices, triangles, two sets of factors per token, the norm's weight
+    int QP, VP8, OP, row_bytes, buf, os, pm, lf, sc, nw, total;
     __host__ __device__ BlockSmem(bool delta, int DP, int VP) {
         QP = DP + 8; VP8 = VP + 8; OP = VP + 4;
         row_bytes = (2 * QP + (delta ? 2 : 1) * VP8) * 2; buf = BM_TB * row_bytes;
-        os = 2 * buf; ph = os + BM_TB * OP * 4; pl = ph + BM_TB * (BM_TB + 8) * 2; mh = pl + BM_TB * (BM_TB + 8) * 2; ml = mh + BM_TB * (BM_TB + 8) * 2;
-        lf = ml + BM_TB * (BM_TB + 8) * 2; sc = lf + BM_TB * 20 * 4; total = sc + 8 * 64 * 4;
+        os = 3 * buf; pm = os + BM_TB * OP * 4; lf = pm + 2 * 4 * BM_PM * 2; sc = lf + BM_TB * 20 * 4; nw = sc + (2 * 6 * BM_TB + 2 * BM_TB) * 4; total = nw + VP * 4;
     }
 };
 
+// A block passes through three stages, each a block ahead of the next: its rows arrive (cp.async), the factors per token and the products of its rows with
+// one another are made, it meets the state.  Per block there are two barriers: between A and B the state's products of block b beside the row products
+// of block b + 1, between B and A the read-outs of block b beside the triangles of block b + 1 and the factors of block b + 2.
 template <bool DELTA, int DP, int THREADS>
 __global__ void __launch_bounds__(THREADS, THREADS == 128 ? 2 : 1) hy_block_memory_kernel(BlockArgs p, HyRows r) {
     HY_PDL();
-    constexpr int NW = THREADS / 32, TPR = THREADS / BM_TB, NT = DP / 8, PP = BM_TB + 8;
+    constexpr int NW = THREADS / 32, TPR = THREADS / BM_TB, NT = DP / 8, PP = BM_PP;
     extern __shared__ __align__(16) uint8_t bm_smem[];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, seq = blockIdx.x, h = blockIdx.y, D = p.D, VD = p.VD, VP = (VD + 15) / 16 * 16;
     const long long row0 = r.seq_row0[seq]; const int len = r.seq_row0[seq + 1] - (int)row0, pos0 = r.seq_pos0[seq];
@@ -57,83 +60,75 @@ __global__ void __launch_bounds__(THREADS, THREADS == 128 ? 2 : 1) hy_block_memo
     const BlockSmem L(DELTA, DP, VP);
     const int QP = L.QP, VP8 = L.VP8, OP = L.OP;
     float* os = reinterpret_cast<float*>(bm_smem + L.os);            // [32][OP] read-outs
-    bf* ph = reinterpret_cast<bf*>(bm_smem + L.ph); bf* pl = reinterpret_cast<bf*>(bm_smem + L.pl);      // [32][PP] e(t, s) q_t . k_s (value, remainder)
-    bf* mh = reinterpret_cast<bf*>(bm_smem + L.mh); bf* ml = reinterpret_cast<bf*>(bm_smem + L.ml);      // [32][PP] inverted triangles on the diagonal, the negated block below
-    float* lf = reinterpret_cast<float*>(bm_smem + L.lf);            // [32][20] the triangles' entries below the diagonal
+    float* lf = reinterpret_cast<float*>(bm_smem + L.lf);            // [32][20] the triangles' entries below the diagonal, column s of a triangle in row s
     float* sc = reinterpret_cast<float*>(bm_smem + L.sc);
-    float *rq = sc, *rk = sc + 64, *Gs = sc + 128, *eG = sc + 192, *wl = sc + 256, *bt = sc + 320, *pw = sc + 384;      // per token: factors of q and k, G, exp(G), e(last, s), beta; powers of a fixed decay
+    float* pw = sc + 12 * BM_TB;                                     // powers of a fixed decay
     const int qh = h / (p.H / p.QH), trow = tid / TPR, tsub = tid % TPR;
     const bf* qg = p.q + row0 * p.ld + (long long)qh * D; const bf* kg = p.k + row0 * p.ld + (long long)qh * D; const bf* vg = p.v + row0 * p.ld + (long long)h * VD;
     const bf* gg = DELTA ? p.gate + row0 * p.ld_in + (long long)h * VD : nullptr;
-    auto Qs = [&](int b) { return reinterpret_cast<bf*>(bm_smem + (b & 1) * L.buf); };
+    const int n_blocks = (len + BM_TB - 1) / BM_TB;
+    auto Qs = [&](int b) { return reinterpret_cast<bf*>(bm_smem + (b % 3) * L.buf); };
     auto Ks = [&](int b) { return Qs(b) + BM_TB * QP; };
     auto Vs = [&](int b) { return Qs(b) + 2 * BM_TB * QP; };
     auto Gt = [&](int b) { return Qs(b) + 2 * BM_TB * QP + BM_TB * VP8; };
-    for (int i = tid; i < 2 * L.buf / 16; i += THREADS) reinterpret_cast<uint4*>(bm_smem)[i] = make_uint4(0, 0, 0, 0);      // padding columns, and rows no block has filled yet
-    float a_next = 0.f, b_next = 0.f;
-    auto fetch = [&](int b) {                            // TPR threads per token, 16 bytes per access
-        const int t = b * BM_TB + trow;
-        if (t < len) {
-            const bf* qr = qg + (long long)t * p.ld; const bf* kr = kg + (long long)t * p.ld; const bf* vr = vg + (long long)t * p.ld;
-            for (int c = tsub * 8; c < D; c += TPR * 8) { cp_async16(Qs(b) + trow * QP + c, qr + c); cp_async16(Ks(b) + trow * QP + c, kr + c); }
-            for (int c = tsub * 8; c < VD; c += TPR * 8) {
-                cp_async16(Vs(b) + trow * VP8 + c, vr + c);
-                if (DELTA) cp_async16(Gt(b) + trow * VP8 + c, gg + (long long)t * p.ld_in + c);
-            }
+    // block matrices, each a value and a remainder [32][PP]: ph | pl e(t, s) q_t . k_s; mh | ml inverted triangles on the diagonal, the negated block below
+    auto ph_of = [&](int b) { return reinterpret_cast<bf*>(bm_smem + L.pm) + (b & 1) * 4 * BM_PM; };
+    auto mh_of = [&](int b) { return ph_of(b) + 2 * BM_PM; };
+    // factors per token: of q and of k, G, exp(G), e(last, s), beta
+    struct Factors { float *rq, *rk, *Gs, *eG, *wl, *bt; };
+    auto factors_of = [&](int b) { float* f = sc + (b & 1) * 6 * BM_TB; return Factors{f, f + BM_TB, f + 2 * BM_TB, f + 3 * BM_TB, f + 4 * BM_TB, f + 5 * BM_TB}; };
+    for (int i = tid; i < 3 * L.buf / 16; i += THREADS) reinterpret_cast<uint4*>(bm_smem)[i] = make_uint4(0, 0, 0, 0);      // padding columns, and rows no block has filled yet
+    for (int i = tid; i < 8 * BM_PM * 2 / 16; i += THREADS) reinterpret_cast<uint4*>(bm_smem + L.pm)[i] = make_uint4(0, 0, 0, 0);      // above the diagonal the matrices stay zero
+    bf a_next = __float2bfloat16_rn(0.f), b_next = a_next;
+    constexpr int QN = DP / 8 / TPR;                     // this thread's 16-byte pieces of a row of q and of k; of v and the gate: two
+    const long long step = (long long)BM_TB * p.ld, step_in = (long long)BM_TB * p.ld_in;
+    const bf *qp = qg + (long long)trow * p.ld + tsub * 8, *kp = kg + (long long)trow * p.ld + tsub * 8, *vp = vg + (long long)trow * p.ld + tsub * 8;
+    const bf *gp = DELTA ? gg + (long long)trow * p.ld_in + tsub * 8 : nullptr, *ap = DELTA ? p.a + (row0 + lane) * p.ld_in + h : nullptr, *bp = DELTA ? p.b + (row0 + lane) * p.ld_in + h : nullptr;
+    auto fetch = [&](int b) {                            // called for b = 0, 1, 2, ...: TPR threads per token, 16 bytes per access
+        if (b * BM_TB + trow < len) {
+            bf* qd = Qs(b) + trow * QP + tsub * 8; bf* vd = Vs(b) + trow * VP8 + tsub * 8;
+#pragma unroll
+            for (int i = 0; i < QN; ++i)
+                if ((tsub + i * TPR) * 8 < D) { cp_async16(qd + i * TPR * 8, qp + i * TPR * 8); cp_async16(qd + BM_TB * QP + i * TPR * 8, kp + i * TPR * 8); }
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+                if ((tsub + i * TPR) * 8 < VD) { cp_async16(vd + i * TPR * 8, vp + i * TPR * 8); if (DELTA) cp_async16(vd + BM_TB * VP8 + i * TPR * 8, gp + i * TPR * 8); }
         }
-        if (DELTA && tid < BM_TB && b * BM_TB + tid < len) {
-            const long long at = (row0 + b * BM_TB + tid) * p.ld_in + h;
-            a_next = ldf(p.a + at); b_next = ldf(p.b + at);
-        }
+        if (DELTA && warp == 0 && b * BM_TB + lane < len) { a_next = *ap; b_next = *bp; }
+        qp += step; kp += step; vp += step;
+        if (DELTA) { gp += step_in; ap += step_in; bp += step_in; }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    __syncthreads();
-    fetch(0);
-    const float al = DELTA ? p.A_log[h] : 0.f, db = DELTA ? p.dt_bias[h] : 0.f;
-    if (!DELTA && tid == 0) { const float d = p.decay[h]; float x = 1.f; for (int i = 0; i <= BM_TB; ++i) { pw[i] = x; x *= d; } }
-    for (int i = tid; i < 2 * BM_TB * PP; i += THREADS) { ph[i] = __float2bfloat16_rn(0.f); mh[i] = __float2bfloat16_rn(0.f); }      // ph | pl and mh | ml lie behind one another; above the diagonal they stay zero
-    // S^T fragments: tile n holds state rows n * 8 + (lane & 3) * 2, + 1 for the value channels v0, v0 + 8
-    const int v0 = warp * 16 + (lane >> 2), dl = (lane & 3) * 2; const bool mine = warp * 16 < VD;
-    float* st = p.state + (((long long)r.seq_state[seq] * p.H + h) * D) * VD;
-    float S[NT][4];
-#pragma unroll
-    for (int n = 0; n < NT; ++n)
-#pragma unroll
-        for (int c = 0; c < 4; ++c) {
-            const int d = n * 8 + dl + (c & 1), vc = v0 + (c >> 1) * 8;
-            S[n][c] = (pos0 > 0 && d < D && vc < VD) ? st[(long long)d * VD + vc] : 0.f;
-        }
-    const float qscale = rsqrtf((float)D);
-    const int brow = (lane >> 4) * 8 + (lane & 7), bcol = ((lane >> 3) & 1) * 8;      // ldmatrix lane addresses of a B operand of 16 rows x 16 columns
-    const int n_blocks = (len + BM_TB - 1) / BM_TB;
-    for (int b = 0; b < n_blocks; ++b) {
-        const int nb = min(BM_TB, len - b * BM_TB);
-        const float a_cur = a_next, b_cur = b_next;
-        asm volatile("cp.async.wait_group 0;" ::: "memory");
-        __syncthreads();                                 // block b has landed; everybody is done with block b - 1
-        if (b + 1 < n_blocks) fetch(b + 1);
-        const bf *Qb = Qs(b), *Kb = Ks(b), *Vb = Vs(b);
+    const float al = DELTA ? p.A_log[h] : 0.f, db = DELTA ? p.dt_bias[h] : 0.f, qscale = rsqrtf((float)D);
+    const int brow = (lane >> 4) * 8 + (lane & 7), bcol = ((lane >> 3) & 1) * 8, dl = (lane & 3) * 2;      // ldmatrix lane addresses of a B operand of 16 rows x 16 columns
+    auto make_factors = [&](int b) {
+        const int nb = min(BM_TB, len - b * BM_TB); const Factors f = factors_of(b);
         if (DELTA) {
+            const bf *Qb = Qs(b), *Kb = Ks(b);
             float sq = 0.f, sk = 0.f;
-            for (int c = tsub * 8; c < D; c += TPR * 8) {
+#pragma unroll
+            for (int i = 0; i < QN; ++i) {               // padding columns are zero
+                const int c = (tsub + i * TPR) * 8;
                 float x[8], y[8];
                 unpack8(*reinterpret_cast<const uint4*>(Qb + trow * QP + c), x); unpack8(*reinterpret_cast<const uint4*>(Kb + trow * QP + c), y);
-#pragma unroll
-                for (int e = 0; e < 8; ++e) { sq = fmaf(x[e], x[e], sq); sk = fmaf(y[e], y[e], sk); }
+                sq += ((x[0] * x[0] + x[1] * x[1]) + (x[2] * x[2] + x[3] * x[3])) + ((x[4] * x[4] + x[5] * x[5]) + (x[6] * x[6] + x[7] * x[7]));
+                sk += ((y[0] * y[0] + y[1] * y[1]) + (y[2] * y[2] + y[3] * y[3])) + ((y[4] * y[4] + y[5] * y[5]) + (y[6] * y[6] + y[7] * y[7]));
             }
 #pragma unroll
             for (int o = 1; o < TPR; o <<= 1) { sq += __shfl_xor_sync(0xffffffffu, sq, o); sk += __shfl_xor_sync(0xffffffffu, sk, o); }
-            if (tsub == 0) { rq[trow] = qscale / sqrtf(sq + 1e-6f); rk[trow] = 1.0f / sqrtf(sk + 1e-6f); }
+            if (tsub == 0) { f.rq[trow] = qscale * rsqrtf(sq + 1e-6f); f.rk[trow] = rsqrtf(sk + 1e-6f); }
             if (warp == 0) {                             // lane = token
-                float G = lane < nb ? log_decay(al, a_cur + db) : 0.f;
+                float G = lane < nb ? log_decay(al, ldf(&a_next) + db) : 0.f;
 #pragma unroll
                 for (int o = 1; o < 32; o <<= 1) { const float u = __shfl_up_sync(0xffffffffu, G, o); if (lane >= o) G += u; }
                 const float Gl = __shfl_sync(0xffffffffu, G, 31);
-                Gs[lane] = G; eG[lane] = expf(G); wl[lane] = lane < nb ? expf(Gl - G) : 0.f; bt[lane] = lane < nb ? sigmoidf_(b_cur) : 0.f;
+                f.Gs[lane] = G; f.eG[lane] = expf(G); f.wl[lane] = lane < nb ? expf(Gl - G) : 0.f; f.bt[lane] = lane < nb ? sigmoidf_(ldf(&b_next)) : 0.f;
             }
-        } else if (tid < BM_TB) { rq[tid] = rk[tid] = 1.f; eG[tid] = pw[tid + 1]; wl[tid] = tid < nb ? pw[nb - 1 - tid] : 0.f; }
-        __syncthreads();
-        // products of the block's rows with one another: units of 16 x 16, the diagonal ones and the one below
+        } else if (tid < BM_TB) { f.rq[tid] = f.rk[tid] = 1.f; f.eG[tid] = pw[tid + 1]; f.wl[tid] = tid < nb ? pw[nb - 1 - tid] : 0.f; }
+    };
+    // products of a block's rows with one another: units of 16 x 16, the diagonal ones and the one below
+    auto row_products = [&](int b) {
+        const bf *Qb = Qs(b), *Kb = Ks(b); const Factors f = factors_of(b); bf *ph = ph_of(b), *mh = mh_of(b);
         for (int u = warp; u < (DELTA ? 6 : 3); u += NW) {
             const bool kk = u >= 3; const int m = (u % 3 + 1) / 2, np = u % 3 == 2 ? 1 : 0;      // (0, 0), (1, 0), (1, 1)
             float acc[2][4] = {};
@@ -144,59 +139,111 @@ __global__ void __launch_bounds__(THREADS, THREADS == 128 ? 2 : 1) hy_block_memo
                 ldmatrix_x4(aa + ks * 32, a0, a1, a2, a3); ldmatrix_x4(ba + ks * 32, b0, b1, b2, b3);
                 mma_bf16_16816(acc[0], a0, a1, a2, a3, b0, b1); mma_bf16_16816(acc[1], a0, a1, a2, a3, b2, b3);
             }
+            // this thread's rows t and columns s, s + 1: their factors first, then the eight entries, stored in pairs
+            const int t0 = m * 16 + (lane >> 2), s0 = np * 16 + dl;
+            float ct[2], gt[2], cs[2][2], gs[2][2];
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                const int t = t0 + i * 8;
+                ct[i] = kk ? f.rk[t] * f.bt[t] : f.rq[t]; gt[i] = DELTA ? f.Gs[t] : 0.f;
+#pragma unroll
+                for (int k = 0; k < 2; ++k) { cs[i][k] = f.rk[s0 + i * 8 + k]; gs[i][k] = DELTA ? f.Gs[s0 + i * 8 + k] : 0.f; }
+            }
 #pragma unroll
             for (int j = 0; j < 2; ++j)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int t = m * 16 + (lane >> 2) + (e >> 1) * 8, s = np * 16 + j * 8 + dl + (e & 1);
-                    if (s > t || (kk && s == t)) continue;
-                    const float f = acc[j][e] * rk[s] * (DELTA ? __expf(Gs[t] - Gs[s]) : pw[t - s]);
-                    if (!kk) split_bf16(f * rq[t], ph[t * PP + s], pl[t * PP + s]);
-                    else if (m == np) lf[t * 20 + s - np * 16] = f * rk[t] * bt[t];
-                    else split_bf16(-f * rk[t] * bt[t], mh[t * PP + s], ml[t * PP + s]);
+                for (int i = 0; i < 2; ++i) {
+                    const int t = t0 + i * 8, s = s0 + j * 8;
+                    float x[2];
+#pragma unroll
+                    for (int k = 0; k < 2; ++k) {
+                        const bool live = kk ? s + k < t : s + k <= t;
+                        x[k] = live ? acc[j][i * 2 + k] * ct[i] * cs[j][k] * (DELTA ? __expf(gt[i] - gs[j][k]) : pw[t - s - k]) : 0.f;
+                    }
+                    if (kk && m == np) { lf[(m * 16 + s - np * 16) * 20 + t - m * 16] = x[0]; lf[(m * 16 + s + 1 - np * 16) * 20 + t - m * 16] = x[1]; }      // column by column
+                    else {
+                        uint32_t hi, lo; split_pack(kk ? -x[0] : x[0], kk ? -x[1] : x[1], hi, lo);
+                        bf* d = (kk ? mh : ph) + t * PP + s;
+                        *reinterpret_cast<uint32_t*>(d) = hi; *reinterpret_cast<uint32_t*>(d + BM_PM) = lo;
+                    }
                 }
         }
-        __syncthreads();
-        if (DELTA && warp == 0) {                        // column lane & 15 of the inverse of triangle lane >> 4
-            const float* lr = lf + (lane >> 4) * 16 * 20; const int c = lane & 15, t0 = (lane >> 4) * 16;
-            float x[16];
+    };
+    auto invert = [&](int b) {                           // one warp: column lane & 15 of the inverse of triangle lane >> 4
+        bf* mh = mh_of(b);
+        const float* lr = lf + (lane >> 4) * 16 * 20; const int c = lane & 15, t0 = (lane >> 4) * 16;
+        float x[16];
 #pragma unroll
-            for (int t = 0; t < 16; ++t) {
-                float s0 = t == c ? 1.f : 0.f, s1 = 0.f;
+        for (int t = 0; t < 16; ++t) x[t] = t == c ? 1.f : 0.f;
 #pragma unroll
-                for (int s = 0; s < t; s += 4) {
-                    const float4 l4 = *reinterpret_cast<const float4*>(lr + t * 20 + s);
-                    s0 = fmaf(-l4.x, x[s], s0);
-                    if (s + 1 < t) s1 = fmaf(-l4.y, x[s + 1], s1);
-                    if (s + 2 < t) s0 = fmaf(-l4.z, x[s + 2], s0);
-                    if (s + 3 < t) s1 = fmaf(-l4.w, x[s + 3], s1);
-                }
-                x[t] = s0 + s1;
-                split_bf16(x[t], mh[(t0 + t) * PP + t0 + c], ml[(t0 + t) * PP + t0 + c]);
+        for (int s = 0; s < 15; ++s)                     // x[s] is final: take it off the rows below
+#pragma unroll
+            for (int q = (s + 1) / 4; q < 4; ++q) {
+                const float4 l4 = *reinterpret_cast<const float4*>(lr + s * 20 + q * 4);
+                if (4 * q > s) x[4 * q] = fmaf(-l4.x, x[s], x[4 * q]);
+                if (4 * q + 1 > s) x[4 * q + 1] = fmaf(-l4.y, x[s], x[4 * q + 1]);
+                if (4 * q + 2 > s) x[4 * q + 2] = fmaf(-l4.z, x[s], x[4 * q + 2]);
+                if (4 * q + 3 > s) x[4 * q + 3] = fmaf(-l4.w, x[s], x[4 * q + 3]);
             }
+#pragma unroll
+        for (int t = 0; t < 16; ++t) split_bf16(x[t], mh[(t0 + t) * PP + t0 + c], mh[BM_PM + (t0 + t) * PP + t0 + c]);
+    };
+    float* nw = reinterpret_cast<float*>(bm_smem + L.nw);
+    if (DELTA) for (int i = tid; i < VD; i += THREADS) nw[i] = p.norm_w[i];
+    if (!DELTA && tid == 0) { const float d = p.decay[h]; float x = 1.f; for (int i = 0; i <= BM_TB; ++i) { pw[i] = x; x *= d; } }
+    __syncthreads();                                     // the buffers are cleared
+    fetch(0);
+    // S^T fragments: tile n holds state rows n * 8 + (lane & 3) * 2, + 1 for the value channels v0, v0 + 8
+    const int v0 = warp * 16 + (lane >> 2); const bool mine = warp * 16 < VD;
+    float* st = p.state + (((long long)r.seq_state[seq] * p.H + h) * D) * VD;
+    float S[NT][4];
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+            const int d = n * 8 + dl + (c & 1), vc = v0 + (c >> 1) * 8;
+            S[n][c] = (pos0 > 0 && d < D && vc < VD) ? st[(long long)d * VD + vc] : 0.f;
         }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    make_factors(0);
+    if (n_blocks > 1) fetch(1);
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    row_products(0);
+    __syncthreads();
+    if (DELTA && warp == NW - 1) invert(0);
+    if (n_blocks > 1) make_factors(1);
+    for (int b = 0; b < n_blocks; ++b) {
+        const int nb = min(BM_TB, len - b * BM_TB);
+        __syncthreads();                                 // A: matrices of block b, factors of block b + 1; everybody is done with block b - 1
+        if (b + 2 < n_blocks) fetch(b + 2);
+        if (b + 1 < n_blocks) row_products(b + 1);
+        const bf *Qb = Qs(b), *Kb = Ks(b), *Vb = Vs(b), *ph = ph_of(b), *pl = ph + BM_PM, *mh = mh_of(b), *ml = mh + BM_PM;
+        const Factors fc = factors_of(b); const float *rq = fc.rq, *rk = fc.rk, *eG = fc.eG, *wl = fc.wl, *bt = fc.bt;
         float kS[4][4] = {}, qS[4][4] = {};              // S^T k and S^T q of the warp's channels: [token tile][..]
         if (mine) {
             const uint32_t ka = smem_u32(Kb + brow * QP + bcol), qa = smem_u32(Qb + brow * QP + bcol);
 #pragma unroll
             for (int ks = 0; ks < DP / 16; ++ks) {
-                uint32_t sh[4], sl[4], b0, b1, b2, b3;
-#pragma unroll
-                for (int i = 0; i < 2; ++i) { split_pack(S[2 * ks + i][0], S[2 * ks + i][1], sh[2 * i], sl[2 * i]); split_pack(S[2 * ks + i][2], S[2 * ks + i][3], sh[2 * i + 1], sl[2 * i + 1]); }
+                uint32_t sh[4], sl[4], kf[2][4], qf[2][4];
 #pragma unroll
                 for (int g = 0; g < 2; ++g) {
-                    if (DELTA) {
-                        ldmatrix_x4(ka + (g * 16 * QP + ks * 16) * 2, b0, b1, b2, b3);
-                        mma_bf16_16816(kS[2 * g], sh[0], sh[1], sh[2], sh[3], b0, b1); mma_bf16_16816(kS[2 * g + 1], sh[0], sh[1], sh[2], sh[3], b2, b3);
-                        mma_bf16_16816(kS[2 * g], sl[0], sl[1], sl[2], sl[3], b0, b1); mma_bf16_16816(kS[2 * g + 1], sl[0], sl[1], sl[2], sl[3], b2, b3);
-                    }
-                    ldmatrix_x4(qa + (g * 16 * QP + ks * 16) * 2, b0, b1, b2, b3);
-                    mma_bf16_16816(qS[2 * g], sh[0], sh[1], sh[2], sh[3], b0, b1); mma_bf16_16816(qS[2 * g + 1], sh[0], sh[1], sh[2], sh[3], b2, b3);
-                    mma_bf16_16816(qS[2 * g], sl[0], sl[1], sl[2], sl[3], b0, b1); mma_bf16_16816(qS[2 * g + 1], sl[0], sl[1], sl[2], sl[3], b2, b3);
+                    if (DELTA) ldmatrix_x4(ka + (g * 16 * QP + ks * 16) * 2, kf[g][0], kf[g][1], kf[g][2], kf[g][3]);
+                    ldmatrix_x4(qa + (g * 16 * QP + ks * 16) * 2, qf[g][0], qf[g][1], qf[g][2], qf[g][3]);
                 }
+#pragma unroll
+                for (int i = 0; i < 2; ++i) { split_pack(S[2 * ks + i][0], S[2 * ks + i][1], sh[2 * i], sl[2 * i]); split_pack(S[2 * ks + i][2], S[2 * ks + i][3], sh[2 * i + 1], sl[2 * i + 1]); }
+                auto pass = [&](const uint32_t (&x)[4]) {        // an accumulator's two products lie a whole pass apart
+#pragma unroll
+                    for (int g = 0; g < 2; ++g) {
+                        if (DELTA) { mma_bf16_16816(kS[2 * g], x[0], x[1], x[2], x[3], kf[g][0], kf[g][1]); mma_bf16_16816(kS[2 * g + 1], x[0], x[1], x[2], x[3], kf[g][2], kf[g][3]); }
+                        mma_bf16_16816(qS[2 * g], x[0], x[1], x[2], x[3], qf[g][0], qf[g][1]); mma_bf16_16816(qS[2 * g + 1], x[0], x[1], x[2], x[3], qf[g][2], qf[g][3]);
+                    }
+                };
+                pass(sh); pass(sl);
             }
         }
-        if (DELTA) __syncthreads();                      // the inverted triangles
         if (mine) {
             // tokens of an accumulator tile n: n * 8 + dl, + 1; of an A operand half g: the tiles 2 g, 2 g + 1
             uint32_t va[2][4];                           // V^T of the warp's channels, in the accumulators' layout
@@ -251,9 +298,24 @@ __global__ void __launch_bounds__(THREADS, THREADS == 128 ? 2 : 1) hy_block_memo
                 const int t = n * 8 + dl; const float f0 = eG[t] * rq[t], f1 = eG[t + 1] * rq[t + 1];
                 qS[n][0] *= f0; qS[n][1] *= f1; qS[n][2] *= f0; qS[n][3] *= f1;
             }
-            times(qS[0], qS[1], uh[0], ul[0], pha + blk(0, 0), pla + blk(0, 0), DELTA);
-            times(qS[2], qS[3], uh[0], ul[0], pha + blk(1, 0), pla + blk(1, 0), DELTA);
-            times(qS[2], qS[3], uh[1], ul[1], pha + blk(1, 1), pla + blk(1, 1), DELTA);
+            {
+                const int tg[3] = {0, 1, 1}, sg[3] = {0, 0, 1};
+                uint32_t f[3][4];
+                auto pass = [&](const uint32_t (&x)[2][4]) {
+#pragma unroll
+                    for (int i = 0; i < 3; ++i) {
+                        mma_bf16_16816(qS[2 * tg[i]], x[sg[i]][0], x[sg[i]][1], x[sg[i]][2], x[sg[i]][3], f[i][0], f[i][1]);
+                        mma_bf16_16816(qS[2 * tg[i] + 1], x[sg[i]][0], x[sg[i]][1], x[sg[i]][2], x[sg[i]][3], f[i][2], f[i][3]);
+                    }
+                };
+#pragma unroll
+                for (int i = 0; i < 3; ++i) ldmatrix_x4(pha + blk(tg[i], sg[i]), f[i][0], f[i][1], f[i][2], f[i][3]);
+                pass(uh);
+                if (DELTA) pass(ul);
+#pragma unroll
+                for (int i = 0; i < 3; ++i) ldmatrix_x4(pla + blk(tg[i], sg[i]), f[i][0], f[i][1], f[i][2], f[i][3]);
+                pass(uh);
+            }
 #pragma unroll
             for (int n = 0; n < 4; ++n)
 #pragma unroll
@@ -271,19 +333,29 @@ __global__ void __launch_bounds__(THREADS, THREADS == 128 ? 2 : 1) hy_block_memo
             const float fS = DELTA ? eG[BM_TB - 1] : pw[nb];
             const uint32_t kt = smem_u32(Kb + (((lane >> 3) & 1) * 8 + (lane & 7)) * QP + (lane >> 4) * 8);
 #pragma unroll
-            for (int n = 0; n < NT; n += 2) {
+            for (int n = 0; n < NT; n += 4) {            // four tiles of state rows at a time: an accumulator's four products lie four apart
+                uint32_t f[2][2][4];
 #pragma unroll
-                for (int e = 0; e < 4; ++e) { S[n][e] *= fS; S[n + 1][e] *= fS; }
+                for (int g = 0; g < 2; ++g)
+#pragma unroll
+                    for (int j = 0; j < 2; ++j) ldmatrix_x4_trans(kt + (g * 16 * QP + (n + 2 * j) * 8) * 2, f[g][j][0], f[g][j][1], f[g][j][2], f[g][j][3]);
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) S[n + j][e] *= fS;
 #pragma unroll
                 for (int g = 0; g < 2; ++g) {
-                    uint32_t b0, b1, b2, b3;
-                    ldmatrix_x4_trans(kt + (g * 16 * QP + n * 8) * 2, b0, b1, b2, b3);
-                    mma_bf16_16816(S[n], uh[g][0], uh[g][1], uh[g][2], uh[g][3], b0, b1); mma_bf16_16816(S[n + 1], uh[g][0], uh[g][1], uh[g][2], uh[g][3], b2, b3);
-                    mma_bf16_16816(S[n], ul[g][0], ul[g][1], ul[g][2], ul[g][3], b0, b1); mma_bf16_16816(S[n + 1], ul[g][0], ul[g][1], ul[g][2], ul[g][3], b2, b3);
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) mma_bf16_16816(S[n + j], uh[g][0], uh[g][1], uh[g][2], uh[g][3], f[g][j >> 1][(j & 1) * 2], f[g][j >> 1][(j & 1) * 2 + 1]);
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) mma_bf16_16816(S[n + j], ul[g][0], ul[g][1], ul[g][2], ul[g][3], f[g][j >> 1][(j & 1) * 2], f[g][j >> 1][(j & 1) * 2 + 1]);
                 }
             }
         }
-        __syncthreads();                                 // the block's read-outs are complete
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();                                 // B: read-outs of block b, triangles of block b + 1, rows of block b + 2
+        if (DELTA && warp == NW - 1 && b + 1 < n_blocks) invert(b + 1);
+        if (b + 2 < n_blocks) make_factors(b + 2);
         const long long trow_g = row0 + b * BM_TB + trow;
         if (DELTA) {
             float x[2][8], ss = 0.f;
@@ -304,7 +376,7 @@ __global__ void __launch_bounds__(THREADS, THREADS == 128 ? 2 : 1) hy_block_memo
                 const int c = (tsub + k * TPR) * 8;
                 if (c < VD && trow < nb) {
                     float g[8], w[8];
-                    unpack8(*reinterpret_cast<const uint4*>(Gt(b) + trow * VP8 + c), g); ld8f(p.norm_w + c, w);
+                    unpack8(*reinterpret_cast<const uint4*>(Gt(b) + trow * VP8 + c), g); ld8f(nw + c, w);
 #pragma unroll
                     for (int e = 0; e < 8; ++e) x[k][e] *= rr * w[e] * silu_fast_f32(g[e]);
                     *reinterpret_cast<uint4*>(reinterpret_cast<bf*>(p.out) + trow_g * p.ldo + (long long)h * VD + c) =
@@ -441,7 +513,7 @@ cudaError_t block_launch(const BlockArgs& p, const HyRows& r, cudaStream_t s) {
     const BlockSmem L(DELTA, DP, VP);
     static bool done[4][16] = {};
     auto go = [&](auto kern, bool (&flag)[16], int threads) -> cudaError_t {
-        if (cudaError_t e = ensure_dynamic_smem(kern, 120 * 1024, flag); e != cudaSuccess) return e;
+        if (cudaError_t e = ensure_dynamic_smem(kern, 160 * 1024, flag); e != cudaSuccess) return e;
         return launch_plain(kern, dim3(r.S, p.H), dim3(threads), (size_t)L.total, s, p, r);
     };
     if (VP <= 64) return DP == 64 ? go(hy_block_memory_kernel<DELTA, 64, 128>, done[0], 128) : go(hy_block_memory_kernel<DELTA, 128, 128>, done[1], 128);

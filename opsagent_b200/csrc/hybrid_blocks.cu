@@ -432,7 +432,7 @@ __global__ void __launch_bounds__(256) hy_few_memory_kernel(FewArgs f, HyRows r)
                 const float x = src >= 0 ? ldf(f.in + (row0 + src) * p.ld_in + ch) : pos0 > 0 ? ldf(tail + (long long)(f.taps - 1 + src) * f.C + ch) : 0.f;
                 acc = fmaf(f.conv_w[ch * f.taps + j], x, acc);
             }
-            *dst = __bfloat162float(__float2bfloat16_rn(siluf_(acc)));      // as the convolution kernel leaves it
+            *dst = __bfloat162float(__float2bfloat16_rn(silu_fast_f32(acc)));      // as the convolution kernel leaves it
         } else *dst = c < D ? ldf(p.q + (row0 + t) * p.ld + (long long)h * D + c) : c < 2 * D ? ldf(p.k + (row0 + t) * p.ld + (long long)h * D + (c - D)) : ldf(p.v + (row0 + t) * p.ld + (long long)h * VD + (c - 2 * D));
     }
     if (tid < len) {

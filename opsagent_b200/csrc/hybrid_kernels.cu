@@ -575,6 +575,20 @@ __global__ void __launch_bounds__(128) hy_gather_ctx_kernel(const __nv_bfloat16*
 // ---------------------------------------------------------------------------------------------------------------------------------
 // short causal convolution with carried tails
 // ---------------------------------------------------------------------------------------------------------------------------------
+// four channels at an aligned place
+__device__ __forceinline__ void ld4(const float* p, float* f) { const float4 u = *reinterpret_cast<const float4*>(p); f[0] = u.x; f[1] = u.y; f[2] = u.z; f[3] = u.w; }
+__device__ __forceinline__ void ld4(const __nv_bfloat16* p, float* f) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    f[0] = __uint_as_float(u.x << 16); f[1] = __uint_as_float(u.x & 0xffff0000u); f[2] = __uint_as_float(u.y << 16); f[3] = __uint_as_float(u.y & 0xffff0000u);
+}
+__device__ __forceinline__ void st4(float* p, const float* f) { *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]); }
+__device__ __forceinline__ void st4(__nv_bfloat16* p, const float* f) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+// SiLU of a value that is stored as the pointer's type: the fast exponential and divide where bf16 rounding follows
+__device__ __forceinline__ float silu_for(float z, const float*) { return siluf_(z); }
+__device__ __forceinline__ float silu_for(float z, const __nv_bfloat16*) { return silu_fast_f32(z); }
 template <typename TA>
 __device__ __forceinline__ float conv_input(const TA* in, int ld_in, int C, const TA* tail, int taps, int row0, int pos0, int src, int c) {
     if (src >= 0) return ldf(in + (long long)(row0 + src) * ld_in + c);
@@ -590,7 +604,7 @@ __global__ void hy_conv_silu_kernel(const TA* in, int ld_in, int C, const float*
     const TA* tail = tails + (long long)r.seq_state[seq] * (taps - 1) * C;
     float acc = bias ? bias[c] : 0.f;
     for (int j = 0; j < taps; ++j) acc = fmaf(w[c * taps + j], conv_input(in, ld_in, C, tail, taps, row0, pos0, i - (taps - 1) + j, c), acc);
-    stf(out + (long long)t * ld_out + c, act ? siluf_(acc) : acc);
+    stf(out + (long long)t * ld_out + c, act ? silu_for(acc, out) : acc);
 }
 // bf16 rows of prefill-sized steps whose channels come in aligned groups of 8: a thread computes 8 channels of CONV_ROWS consecutive rows
 // from 16-byte loads, with its taps' weights and the last inputs in registers, so that every input row is read once.  The sum runs over
@@ -605,20 +619,30 @@ template <int TAPS>
 __global__ void __launch_bounds__(128) hy_conv_silu_vec8_kernel(const __nv_bfloat16* __restrict__ in, int ld_in, int C, const float* __restrict__ w, const float* __restrict__ bias,
                                                                  __nv_bfloat16* __restrict__ out, int ld_out, const __nv_bfloat16* __restrict__ tails, HyRows r, int act) {
     HY_PDL();
-    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8, t0 = blockIdx.y * CONV_ROWS;
+    // the block's row metadata once, in shared memory, and input rows requested ahead: a thread's chain per row is arithmetic only
+    __shared__ int s_row0[CONV_ROWS], s_pos0[CONV_ROWS], s_state[CONV_ROWS];
+    const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8, t0 = blockIdx.y * CONV_ROWS, n = min(CONV_ROWS, r.T - t0);
+    if (threadIdx.x < n) { const int seq = r.row_seq[t0 + threadIdx.x]; s_row0[threadIdx.x] = r.seq_row0[seq]; s_pos0[threadIdx.x] = r.seq_pos0[seq]; s_state[threadIdx.x] = r.seq_state[seq]; }
+    __syncthreads();
     if (c >= C) return;
-    float wr[TAPS][8], win[TAPS][8], b8[8];
+    constexpr int AHEAD = 4;
+    uint4 ring[AHEAD];
 #pragma unroll
-    for (int e = 0; e < 8; ++e) {
-        b8[e] = bias ? bias[c + e] : 0.f;
+    for (int k = 0; k < AHEAD; ++k) if (k < n) ring[k] = *reinterpret_cast<const uint4*>(in + (long long)(t0 + k) * ld_in + c);
+    float wf[8 * TAPS], win[TAPS][8], b8[8];             // taps of the thread's channels, [channel][tap] as they lie
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) wr[j][e] = w[(c + e) * TAPS + j];
-    }
-    for (int tt = 0; tt < CONV_ROWS && t0 + tt < r.T; ++tt) {
-        const int t = t0 + tt, seq = r.row_seq[t], row0 = r.seq_row0[seq], i = t - row0;
+    for (int i = 0; i < 2 * TAPS; ++i) ld4(w + (long long)c * TAPS + i * 4, wf + i * 4);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) b8[e] = bias ? bias[c + e] : 0.f;
+#pragma unroll
+    for (int tt = 0; tt < CONV_ROWS; ++tt) {
+        if (tt >= n) break;
+        const int t = t0 + tt, row0 = s_row0[tt], i = t - row0;
+        const uint4 cur = ring[tt % AHEAD];
+        if (tt + AHEAD < n) ring[tt % AHEAD] = *reinterpret_cast<const uint4*>(in + (long long)(t + AHEAD) * ld_in + c);
         if (tt == 0 || i == 0) {                        // the inputs before this row: earlier rows of the step, the carried tail, or zeros
-            const int pos0 = r.seq_pos0[seq];
-            const __nv_bfloat16* tail = tails + (long long)r.seq_state[seq] * (TAPS - 1) * C;
+            const int pos0 = s_pos0[tt];
+            const __nv_bfloat16* tail = tails + (long long)s_state[tt] * (TAPS - 1) * C;
 #pragma unroll
             for (int j = 0; j < TAPS - 1; ++j) {
                 const int src = i - (TAPS - 1) + j;
@@ -628,17 +652,16 @@ __global__ void __launch_bounds__(128) hy_conv_silu_vec8_kernel(const __nv_bfloa
                 bf8_to_f32(u, win[j]);
             }
         }
-        bf8_to_f32(*reinterpret_cast<const uint4*>(in + (long long)t * ld_in + c), win[TAPS - 1]);
-        uint32_t o[4];
+        bf8_to_f32(cur, win[TAPS - 1]);
+        float o[8];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            float a0 = b8[2 * e], a1 = b8[2 * e + 1];
+        for (int e = 0; e < 8; ++e) {
+            float a = b8[e];
 #pragma unroll
-            for (int j = 0; j < TAPS; ++j) { a0 = fmaf(wr[j][2 * e], win[j][2 * e], a0); a1 = fmaf(wr[j][2 * e + 1], win[j][2 * e + 1], a1); }
-            const __nv_bfloat162 h = act ? __floats2bfloat162_rn(siluf_(a0), siluf_(a1)) : __floats2bfloat162_rn(a0, a1);
-            o[e] = *reinterpret_cast<const uint32_t*>(&h);
+            for (int j = 0; j < TAPS; ++j) a = fmaf(wf[e * TAPS + j], win[j][e], a);
+            o[e] = act ? silu_for(a, out) : a;
         }
-        *reinterpret_cast<uint4*>(out + (long long)t * ld_out + c) = make_uint4(o[0], o[1], o[2], o[3]);
+        *reinterpret_cast<uint4*>(out + (long long)t * ld_out + c) = make_uint4(pack_bf16x2(o[0], o[1]), pack_bf16x2(o[2], o[3]), pack_bf16x2(o[4], o[5]), pack_bf16x2(o[6], o[7]));
 #pragma unroll
         for (int j = 0; j < TAPS - 1; ++j)
 #pragma unroll
@@ -886,16 +909,6 @@ __global__ void __launch_bounds__(128) hy_gated_norm_kernel(const float* o, int 
 
 // The same for groups that one warp handles well (prefill-sized steps): a warp per (row, group), four consecutive channels per lane and
 // step, no block barrier.  The second pass re-reads what the first left in L1.
-__device__ __forceinline__ void ld4(const float* p, float* f) { const float4 u = *reinterpret_cast<const float4*>(p); f[0] = u.x; f[1] = u.y; f[2] = u.z; f[3] = u.w; }
-__device__ __forceinline__ void ld4(const __nv_bfloat16* p, float* f) {
-    const uint2 u = *reinterpret_cast<const uint2*>(p);
-    f[0] = __uint_as_float(u.x << 16); f[1] = __uint_as_float(u.x & 0xffff0000u); f[2] = __uint_as_float(u.y << 16); f[3] = __uint_as_float(u.y & 0xffff0000u);
-}
-__device__ __forceinline__ void st4(float* p, const float* f) { *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]); }
-__device__ __forceinline__ void st4(__nv_bfloat16* p, const float* f) {
-    const __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
-    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
-}
 template <typename TA>
 __global__ void __launch_bounds__(128) hy_gated_norm_warp_kernel(const float* __restrict__ o, int C, int group, const float* __restrict__ w, int wlen, const TA* __restrict__ gate,
                                                                   int ld_gate, int gate_before, int act, const float* __restrict__ skip, int skip_block, const TA* __restrict__ xs,
@@ -1369,7 +1382,7 @@ cudaError_t hy_mha_prefill(const HyLatentAttn& a, const void* q, int ldq, const 
 cudaError_t hy_conv_silu(bool f32, const void* in, int ld_in, int C, const float* w, const float* bias, int taps, void* out, int ld_out, const void* tails, const HyRows& r,
                          cudaStream_t s, int act) {
     auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-    if (!f32 && r.T >= 512 && taps >= 2 && taps <= 4 && C % 8 == 0 && ld_in % 8 == 0 && ld_out % 8 == 0 && al16(in) && al16(out) && al16(tails)) {
+    if (!f32 && r.T >= 512 && taps >= 2 && taps <= 4 && C % 8 == 0 && ld_in % 8 == 0 && ld_out % 8 == 0 && al16(in) && al16(out) && al16(tails) && al16(w)) {
         const dim3 g((C / 8 + 127) / 128, (r.T + CONV_ROWS - 1) / CONV_ROWS);
         switch (taps) {
             case 2: return launch_plain(hy_conv_silu_vec8_kernel<2>, g, dim3(128), 0, s, (const bf*)in, ld_in, C, w, bias, (bf*)out, ld_out, (const bf*)tails, r, act);

@@ -586,9 +586,11 @@ __device__ __forceinline__ void st4(__nv_bfloat16* p, const float* f) {
     const __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
     *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
 }
-// SiLU of a value that is stored as the pointer's type: the fast exponential and divide where bf16 rounding follows
+// SiLU / sigmoid of a value that is stored as the pointer's type: the fast exponential and divide where bf16 rounding follows
 __device__ __forceinline__ float silu_for(float z, const float*) { return siluf_(z); }
 __device__ __forceinline__ float silu_for(float z, const __nv_bfloat16*) { return silu_fast_f32(z); }
+__device__ __forceinline__ float sigmoid_for(float z, const float*) { return sigmoidf_(z); }
+__device__ __forceinline__ float sigmoid_for(float z, const __nv_bfloat16*) { return __fdividef(1.0f, 1.0f + __expf(-z)); }
 template <typename TA>
 __device__ __forceinline__ float conv_input(const TA* in, int ld_in, int C, const TA* tail, int taps, int row0, int pos0, int src, int c) {
     if (src >= 0) return ldf(in + (long long)(row0 + src) * ld_in + c);
@@ -955,7 +957,7 @@ __global__ void __launch_bounds__(128) hy_gated_norm_warp_kernel(const float* __
     }
 }
 
-// Groups too wide for a warp (gate behind the norm, or none): one CTA per (row, group), the group's values in registers, 16-byte accesses
+// Groups too wide for a warp (gate behind the norm, or none; one weight for all groups or one per channel): one CTA per (row, group), the group's values in registers, 16-byte accesses
 template <typename TA, int NV>      // NV x 4 channels per thread: group <= 1024 NV
 __global__ void __launch_bounds__(256) hy_gated_norm_wide_kernel(const float* __restrict__ o, int C, int group, const float* __restrict__ w, int wlen, const TA* __restrict__ gate, int ld_gate, int act,
                                                                  TA* __restrict__ out, int ld_out, float eps) {
@@ -977,10 +979,12 @@ __global__ void __launch_bounds__(256) hy_gated_norm_wide_kernel(const float* __
     for (int k = 0; k < NV; ++k) {
         const int i = (threadIdx.x + k * 256) * 4;
         if (i >= group) continue;
+        float wv[4] = {1.f, 1.f, 1.f, 1.f};
+        if (w) ld4(w + (wlen == group ? i : c0 + i), wv);
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            v[k][e] *= rr * (w ? w[(c0 + i + e) % wlen] : 1.f);
-            if (gate) v[k][e] *= act ? siluf_(g[k][e]) : sigmoidf_(g[k][e]);
+            v[k][e] *= rr * wv[e];
+            if (gate) v[k][e] *= act ? silu_for(g[k][e], out) : sigmoid_for(g[k][e], out);
         }
         st4(out + t * ld_out + c0 + i, v[k]);
     }
@@ -1457,7 +1461,7 @@ cudaError_t hy_gated_norm(bool f32, const float* o, int C, int group, const floa
                    : launch_plain(hy_gated_norm_warp_kernel<bf>, g, dim3(128), 0, s, o, C, group, w, wlen, (const bf*)gate, ld_gate, gate_before, act, skip, skip_block, (const bf*)xs, ld_xs, (bf*)out, ld_out, eps, n, den_dot, den_floor);
     }
     dim3 grid(T, C / group);
-    if (group % 4 == 0 && group > 512 && group <= 8192 && !skip && !den_dot && !(gate && gate_before) && C % 4 == 0 && ld_gate % 4 == 0 && ld_out % 4 == 0 && al(o, 16) && al(gate, 4 * ea) && al(out, 4 * ea)) {
+    if (group % 4 == 0 && group > 512 && group <= 8192 && !skip && !den_dot && !(gate && gate_before) && (!w || ((wlen == group || wlen == C) && al(w, 16))) && C % 4 == 0 && ld_gate % 4 == 0 && ld_out % 4 == 0 && al(o, 16) && al(gate, 4 * ea) && al(out, 4 * ea)) {
 #define HY_GNW(NV) (f32 ? launch_plain(hy_gated_norm_wide_kernel<float, NV>, grid, dim3(256), 0, s, o, C, group, w, wlen, (const float*)gate, ld_gate, act, (float*)out, ld_out, eps) \
                         : launch_plain(hy_gated_norm_wide_kernel<bf, NV>, grid, dim3(256), 0, s, o, C, group, w, wlen, (const bf*)gate, ld_gate, act, (bf*)out, ld_out, eps))
         return group <= 1024 ? HY_GNW(1) : group <= 2048 ? HY_GNW(2) : group <= 4096 ? HY_GNW(4) : HY_GNW(8);

@@ -1,4 +1,4 @@
-// hybrid_kernels.hpp — launch API of the kernels behind the hybrid decoder family (hybrid_kernels.cu, hybrid_window.cu, hybrid_linear.cu, hybrid_streams.cu): layer norm and RMS
+// hybrid_kernels.hpp — launch API of the kernels behind the hybrid decoder family (hybrid_kernels.cu, hybrid_window.cu, hybrid_linear.cu, hybrid_blocks.cu, hybrid_streams.cu): layer norm and RMS
 // norm, latent attention over a paged latent cache, windowed attention over paged keys and values (sliding window, kept first tokens,
 // differential maps, sink, output gates, soft cap and distance slope on the scores, a norm over the whole projection, a query temperature),
 // causal short convolutions with carried tails, the linear recurrences (gated delta rule with per-channel decay, Mamba-2, gated linear
@@ -10,6 +10,7 @@
 // Norms on both sides of a sublayer, PolyNorm (hybrid_streams.cu); a learned bias per distance on the scores, unit-RMS values mixed with another
 // layer's (hybrid_window.cu); the recurrence that writes with the complement of its forget gate, alone and fused with its gates and its norm
 // (hybrid_linear.cu); a router of plain sigmoids and experts with a clamped gated activation and a weight on their input (hybrid_kernels.cu).
+// Recurrences with one decay per head — lightning attention, the gated delta rule — from projections to heads' outputs in one kernel (hybrid_blocks.cu).
 // Each mechanism takes its sizes and constants as arguments.
 //
 // `f32` selects the activation / matrix element type: false = bf16 storage with fp32 accumulation, true = everything in fp32.  What must be
@@ -103,7 +104,7 @@ cudaError_t hy_win_prep(bool f32, const HyWinAttn& a, void* q, int ldq, const vo
 cudaError_t hy_win_attention(bool f32, const HyWinAttn& a, const void* q, int ldq, const void* cache, const float* sink, const void* gate, int ldg, void* out, int ldo, float eps,
                              const HyRows& r, cudaStream_t s);
 
-// tensor-core form (bf16; dim a multiple of 16 up to 128, vdim 16 / 32 / 64 / 96 / 128), for prompt portions and decoding rows alike: a tile =
+// tensor-core form (bf16; dim a multiple of 16 up to 128, vdim 16 / 32 / 64 / 96 / 128, with score modifiers also 48 / 80), for prompt portions and decoding rows alike: a tile =
 // 64 consecutive (row, head-of-the-group) pairs of one sequence starting at pair tile_q0 (pair p = row p / group, head p % group of the
 // CTA's key/value head, group = heads / kv_heads); grid = tiles x kv_heads.  The host lists the tiles of a step.
 constexpr int HY_WIN_TILE_QUERIES = 64;
